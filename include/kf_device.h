@@ -48,6 +48,7 @@ enum {
                           int32 [cols / 128][rows / 8], step_dev = scales fp16 [cols / 128][rows]; w = bf16(float(q - z) * scale)
                           (CU_Q42X_awq, quantizer.cu:132-156; CU_I2Q4_unpack, packedN.cuh:109-116).  rows = out_features, cols =
                           in_features, group = 128.  Device-level only: kf_dequant / kf_linear*; no quantiser (vendor checkpoints)   */
+    KF_T_I32      = 8, /* a table of 32-bit integers (ids); storage only: no matmul, no quantiser, no dequantiser                    */
 };
 
 /* ---- quantisation modes (QUANT_CARD, src/CLI_params.hpp:509-554; GeQuant ctor src/Tensor/GeQuant.cpp:107-124) ---- */
@@ -415,6 +416,52 @@ int kf_latent_attention_ex(kf_ctx* ctx, float* lat_out_dev, float* qa_work_dev, 
                            const void* sink_bf16_dev, const void* cache_dev, int cache_f32, size_t slot_stride, const double* inv_freq_dev,
                            const int32_t* pos_dev, const int32_t* slot_dev, int M, int H, int dn, int rot_dim, int rot_dims, int rank, float scale,
                            int max_pos_hint, int layout, float amp);
+
+/* ---- post-norm stacks with shifted inputs, windowed attention beside pooled blocks of positions, experts named by a table of token ids
+ *      (ops_f32.cu, attn_window.cu, attention.cu); no reference equivalents ---- */
+/* kf_postnorm_residual with a factor on what is added (mult), a norm weight that may be one number (w_one 1), and -- when every row is one token
+ * of a sequence of its own -- the token shift of the next sublayer's input folded in: act_out = x + (prev - x) * shift, prev = the sequence's
+ * tail [slot][tail_stride] (zeros at position 0), which then takes x (shift_bf16 [dim] NULL: act_out = x) */
+int kf_postnorm_residual_ex(kf_ctx* ctx, float* res_dev, void* act_out_dev, int act_f32, const float* a_dev, int lda, float sa, const float* b_dev, int ldb, float sb,
+                            const void* w_bf16_dev, float w_add, int w_one, float mult, int rows, int dim, float eps, const void* shift_bf16_dev, float* tail_dev,
+                            size_t tail_stride, const int32_t* pos_dev, const int32_t* slot_dev);
+/* the same step over the sum of a token's experts, sum_j wgt[m][j] * y_slots[entry_slot[m][j]] (+ shared[m]) */
+int kf_experts_postnorm_residual(kf_ctx* ctx, float* res_dev, void* act_out_dev, int act_f32, const float* y_slots_dev, const int32_t* entry_slot_dev,
+                                 const float* wgt_dev, const float* shared_dev, int top, const void* w_bf16_dev, float w_add, int w_one, float mult, int rows, int dim,
+                                 float eps, const void* shift_bf16_dev, float* tail_dev, size_t tail_stride, const int32_t* pos_dev, const int32_t* slot_dev);
+/* res[m] = rmsnorm(W[token[m]]) * (w_add + w); act_out and shift as above */
+int kf_embed_norm(kf_ctx* ctx, float* res_dev, void* act_out_dev, int act_f32, const kf_tensor_desc* table, const int32_t* tokens_dev, const void* w_bf16_dev,
+                  float w_add, int w_one, int rows, float eps, const void* shift_bf16_dev, float* tail_dev, size_t tail_stride, const int32_t* pos_dev,
+                  const int32_t* slot_dev);
+/* out[t] = h[t] + (h[t-1] - h[t]) * w over nseq sequences of T consecutive rows, in the activation type; h[-1] from the slot's tail (zeros at
+ * position 0), which takes the last row */
+int kf_token_shift(kf_ctx* ctx, void* out_dev, int out_f32, const float* h_dev, int ldh, const void* w_bf16_dev, float* tail_dev, size_t tail_stride,
+                   const int32_t* pos_dev, const int32_t* slot_dev, int nseq, int T, int dim);
+/* routing from a table of token ids (int32 [vocab][top], the experts of each token; weights 1 / top): the dispatch tables of kf_moe_route for
+ * n_routes layers in one go; routes_dev: device array of n_routes entries; work: M * top + experts ints */
+typedef struct kf_table_route {
+    const int32_t* table;
+    int32_t *idx, *offsets, *entry_slot, *slot_row, *slot_group, *work;
+    float* wgt;
+    int experts, top;
+} kf_table_route;
+int kf_moe_route_table(kf_ctx* ctx, const kf_table_route* routes_dev, int n_routes, int max_experts, int max_top, const int32_t* tokens_dev, int M);
+/* x[m] = [q (H x dk) | k (G x dk) | v (G x dv)] floats: RMS norm of every head of q and k on its own (weights bf16 [dk] shared by the heads, NULL:
+ * none), rotation as kf_qk_prepare (rot_dims 0: none), k | v into row pos % ring of the slot's cache; q in place, or as bf16 into q_bf16_out.
+ * pool > 0: a token that completes a block of `pool` positions makes row ring + block of its slot the mean of the block's rows.
+ * one_per_slot 1: the M tokens belong to M different slots */
+int kf_qk_heads_prepare(kf_ctx* ctx, float* x_dev, int ldx, int H, int G, int dk, int dv, const void* q_norm_bf16_dev, const void* k_norm_bf16_dev, float eps,
+                        int rot_dims, const double* inv_freq_dev, float amp, int layout, void* cache_dev, int cache_f32, size_t slot_stride, int ring, int pool,
+                        int one_per_slot, void* q_bf16_out_dev, const int32_t* pos_dev, const int32_t* slot_dev, int M);
+/* kf_attn_window with pooled blocks (pool > 0: token m also sees row ring + b of every block b with b * pool + pool - 1 <= pos[m] - window, in the
+ * same softmax) and a gate per head (the result of head h times sigmoid(head_gate[m * ldg + h]), NULL: none) */
+int kf_attn_window_ex(kf_ctx* ctx, void* out_dev, int out_f32, int ldo, const float* q_dev, int ldq, const void* cache_dev, int cache_f32, size_t slot_stride,
+                      int ring, const void* sink_bf16_dev, const int32_t* pos_dev, const int32_t* slot_dev, int M, int H, int G, int dk, int dv, float scale,
+                      float softcap, int window, int max_keys_hint, float out_scale, int pool, const float* head_gate_dev, int ldg);
+/* the same attention for a panel of M consecutive tokens of one slot on the tensor cores (bf16 ring cache, dk == dv in {64, 128}; attention.cu) */
+int kf_attn_pooled_prefill(kf_ctx* ctx, void* out_bf16_dev, int ldo, const void* q_bf16_dev, const void* cache_dev, size_t slot_stride, int ring,
+                           const void* sink_bf16_dev, const int32_t* pos_dev, const int32_t* slot_dev, int M, int n_head, int n_kv, int hd, float scale,
+                           float softcap, int window, int pool, const float* head_gate_dev, int ldg, float out_scale);
 
 #ifdef __cplusplus
 }

@@ -43,6 +43,8 @@ int kf_model_init_random(kf_model* m);
 /* SERIALIZE path: hand over one FULL (unsharded) bf16 tensor by its HF name (NN2NAME, src/Transformer/QWen.cpp:61-145);
  * it is sharded for this rank and quantised at load */
 int kf_model_set_tensor(kf_model* m, const char* hf_name, const void* host_bf16, int rows, int cols);
+/* hand over a tensor that is a table of 32-bit ids (full shape; every id is checked against the model's limit) */
+int kf_model_set_tensor_i32(kf_model* m, const char* hf_name, const int32_t* host_i32, int rows, int cols);
 /* One linear of a vendor-quantised (AWQ) checkpoint by the HF name of its weight ("....q_proj.weight"), FULL shape, in the arrays the
  * checkpoint stores (GeQuant::ExTensor src/Tensor/GeQuant.cpp:144-200, GTensor::LoadParam src/Manifold/Serialize.cpp:145-230, unpack
  * CU_Q42X_awq src/Device/CUDA/kernel/quantizer.cu:132-156): qweight int32 [in][out / 8] (nibbles in AWQ_REVERSE_ORDER), qzeros int32

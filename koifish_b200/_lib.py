@@ -143,6 +143,14 @@ SIGNATURES = {
     "kf_attn_sigmoid_prefill": (_I, [_P, _P, _I, _P, _P, _SZ, _I, _P, _P, _P, _I, _I, _I, _I, _F, _I, _F]),
     "kf_latent_append_ex": (_I, [_P, _P, _I, _SZ, _P, _I, _P, _P, _P, _P, _I, _I, _I, _I, _F, _I, _F]),
     "kf_latent_attention_ex": (_I, [_P, _P, _P, _P, _I, _P, _P, _P, _I, _SZ, _P, _P, _P, _I, _I, _I, _I, _I, _I, _F, _I, _I, _F]),
+    "kf_postnorm_residual_ex": (_I, [_P, _P, _P, _I, _P, _I, _F, _P, _I, _F, _P, _F, _I, _F, _I, _I, _F, _P, _P, _SZ, _P, _P]),
+    "kf_experts_postnorm_residual": (_I, [_P, _P, _P, _I, _P, _P, _P, _P, _I, _P, _F, _I, _F, _I, _I, _F, _P, _P, _SZ, _P, _P]),
+    "kf_embed_norm": (_I, [_P, _P, _P, _I, _DESCP, _P, _P, _F, _I, _I, _F, _P, _P, _SZ, _P, _P]),
+    "kf_token_shift": (_I, [_P, _P, _I, _P, _I, _P, _P, _SZ, _P, _P, _I, _I, _I]),
+    "kf_moe_route_table": (_I, [_P, _P, _I, _I, _I, _P, _I]),
+    "kf_qk_heads_prepare": (_I, [_P, _P, _I, _I, _I, _I, _I, _P, _P, _F, _I, _P, _F, _I, _P, _I, _SZ, _I, _I, _I, _P, _P, _P, _I]),
+    "kf_attn_window_ex": (_I, [_P, _P, _I, _I, _P, _I, _P, _I, _SZ, _I, _P, _P, _P, _I, _I, _I, _I, _I, _F, _F, _I, _I, _F, _I, _P, _I]),
+    "kf_attn_pooled_prefill": (_I, [_P, _P, _I, _P, _P, _SZ, _I, _P, _P, _P, _I, _I, _I, _I, _F, _F, _I, _I, _P, _I, _F]),
     "kf_nccl_unique_id": (_I, [_P]),
     "kf_ctx_init_nccl": (_I, [_P, _P, _I, _I]),
     "kf_allreduce_bf16": (_I, [_P, _P, _SZ]),
@@ -156,6 +164,7 @@ SIGNATURES = {
     "kf_model_info_get": (_I, [_P, C.POINTER(ModelInfo)]),
     "kf_model_init_random": (_I, [_P]),
     "kf_model_set_tensor": (_I, [_P, C.c_char_p, _P, _I, _I]),
+    "kf_model_set_tensor_i32": (_I, [_P, C.c_char_p, _P, _I, _I]),
     "kf_model_set_tensor_awq": (_I, [_P, C.c_char_p, _P, _P, _P, _I, _I]),
     "kf_model_tensor_desc": (_I, [_P, C.c_char_p, _DESCP]),
     "kf_model_tensor_count": (_I, [_P]),

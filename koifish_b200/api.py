@@ -416,6 +416,12 @@ class Model:
         self._check(self.lib.kf_model_init_random(self.h), "kf_model_init_random")
 
     def set_tensor(self, name, w_bf16):
+        """bf16 bit patterns (uint16), or, for a tensor that is a table of ids, int32 values"""
+        if np.asarray(w_bf16).dtype == np.int32:
+            ids = np.ascontiguousarray(w_bf16)
+            rows, cols = (1, ids.size) if ids.ndim == 1 else ids.shape
+            self._check(self.lib.kf_model_set_tensor_i32(self.h, name.encode(), ids.ctypes.data, rows, cols), "kf_model_set_tensor_i32(%s)" % name)
+            return
         w = np.ascontiguousarray(w_bf16, dtype=np.uint16)
         rows, cols = (1, w.size) if w.ndim == 1 else w.shape
         self._check(self.lib.kf_model_set_tensor(self.h, name.encode(), w.ctypes.data, rows, cols), "kf_model_set_tensor(%s)" % name)

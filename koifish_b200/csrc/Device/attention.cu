@@ -566,16 +566,21 @@ struct PfBias {
     // weights are not normalised over the keys
     int block;
     const uint16_t* hbias;
+    // MODE 4 (MODE 2 with pooled blocks and a gate per head): a query at p also sees the rows ring + b of the blocks b of `pool` positions with
+    // b * pool + pool - 1 <= p - window (pool 0: none); the result of head h times sigmoid(hgate[row * ldg + h]) (NULL: not)
+    int pool;
+    const float* hgate;
 };
 // MODE 0: Qwen3's plain causal attention over separate K and V caches.  MODE 1: see above.  MODE 2: the side-by-side rows and hi + lo
 // softmax weights of MODE 1 without penalty and gate, with the window, cap, sink and ring of PfBias.  MODE 3: the rows and the ring of
-// MODE 2 with sigmoid weights inside blocks of positions -- no running maximum, no rescaling, no denominator.
+// MODE 2 with sigmoid weights inside blocks of positions -- no running maximum, no rescaling, no denominator.  MODE 4: MODE 2 over pooled
+// blocks as well, whose tiles come ahead of the window's.
 template <int HD, int BKV, int MODE>
 __global__ void __launch_bounds__(128, KF_PF_MINB) kf_attn_prefill_kernel(uint16_t* __restrict__ out, const uint16_t* __restrict__ q,
                                                               const uint16_t* __restrict__ kc, const uint16_t* __restrict__ vc,
                                                               const int32_t* __restrict__ pos_dev, int M, int n_head, int n_kv, int max_seq,
                                                               float sqrt_hd, PfBias xb) {
-    constexpr bool BIAS = MODE == 1, WIN = MODE == 2, SIG = MODE == 3, RING = MODE >= 2, ROWS = MODE != 0;
+    constexpr bool BIAS = MODE == 1, WIN = MODE == 2 || MODE == 4, SIG = MODE == 3, POOL = MODE == 4, RING = MODE >= 2, ROWS = MODE != 0;
     constexpr int CH = HD / 8;  // 16-byte chunks per row
     extern __shared__ __align__(16) uint8_t pf_smem[];
     const uint32_t sQ = (uint32_t)__cvta_generic_to_shared(pf_smem);
@@ -592,6 +597,8 @@ __global__ void __launch_bounds__(128, KF_PF_MINB) kf_attn_prefill_kernel(uint16
     const int ntiles = (kv_len + BKV - 1) / BKV;
     // the first tile that the tile's first query still sees
     const int kt0 = WIN ? max(0, pos0 + q0 - xb.window + 1) / BKV : SIG ? (((pos0 + q0) / xb.block) * xb.block) / BKV : 0;
+    // pooled tiles: blocks 0 .. nb_max - 1 are those that the tile's last query sees; tile indices below kt0 stand for them
+    const int nb_max = (POOL && xb.pool > 0) ? max(0, kv_len - xb.window) / xb.pool : 0, npt = POOL ? (nb_max + BKV - 1) / BKV : 0, it0 = kt0 - npt;
     const float hb2 = (SIG && xb.hbias) ? bf16_bits_to_f32(xb.hbias[h]) * 1.4426950408889634f : 0.f;
     // where the blocks of this thread's two query rows start
     const int b_lo = SIG ? ((pos0 + q0 + (threadIdx.x >> 5) * 16 + ((threadIdx.x & 31) >> 2)) / xb.block) * xb.block : 0;
@@ -608,12 +615,12 @@ __global__ void __launch_bounds__(128, KF_PF_MINB) kf_attn_prefill_kernel(uint16
         for (int i = tid; i < BKV * CH; i += 128) {
             const int r = i / CH, c = i % CH;
             // rows past kv_len are masked below; keep the address inside the cache (WIN: any row of the ring will do for those)
-            const int t = RING ? (kt * BKV + r) % xb.ring : min(kt * BKV + r, max_seq - 1);
+            const int t = (POOL && kt < kt0) ? xb.ring + min((kt - it0) * BKV + r, nb_max - 1) : RING ? (kt * BKV + r) % xb.ring : min(kt * BKV + r, max_seq - 1);
             cp16(sK + buf * (BKV * HD * 2) + sw(r, c), kc + (size_t)t * kv_dim + (size_t)kvh * HD + c * 8, true);
             cp16(sV + buf * (BKV * HD * 2) + sw(r, c), vc + (size_t)t * kv_dim + (size_t)kvh * HD + c * 8, true);
         }
     };
-    load_kv(kt0, kt0 & 1);
+    load_kv(it0, it0 & 1);
     asm volatile("cp.async.commit_group;" ::: "memory");
 
     uint32_t qa[HD / 16][4];
@@ -622,17 +629,18 @@ __global__ void __launch_bounds__(128, KF_PF_MINB) kf_attn_prefill_kernel(uint16
     for (int j = 0; j < HD / 8; j++) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
     float m_lo = -INFINITY, m_hi = -INFINITY, l_lo = 0.f, l_hi = 0.f;
     const int p_lo = pos0 + q0 + warp * 16 + g, p_hi = p_lo + 8;  // positions of this thread's two query rows
+    const int nb_lo = (POOL && xb.pool > 0) ? max(0, p_lo - xb.window + 1) / xb.pool : 0, nb_hi = (POOL && xb.pool > 0) ? max(0, p_hi - xb.window + 1) / xb.pool : 0;
     // softmax((q.k)/sqrt(hd)) = 2^((q.k - max) * log2(e)/sqrt(hd)) / sum ; BIAS: the scores are brought to the log2 domain where the penalty joins
     const float SC = ROWS ? 1.f : 1.4426950408889634f / sqrt_hd, SCB = xb.scale * 1.4426950408889634f;
     const float cap2 = (WIN && xb.softcap > 0.f) ? 2.f * 1.4426950408889634f / xb.softcap : 0.f, capL = xb.softcap * 1.4426950408889634f;
 
-    for (int kt = kt0; kt < ntiles; kt++) {
+    for (int kt = it0; kt < ntiles; kt++) {
         const int buf = kt & 1;
         if (kt + 1 < ntiles) load_kv(kt + 1, buf ^ 1);
         asm volatile("cp.async.commit_group;" ::: "memory");
         asm volatile("cp.async.wait_group 1;" ::: "memory");
         __syncthreads();
-        if (kt == kt0) {
+        if (kt == it0) {
 #pragma unroll
             for (int kc_ = 0; kc_ < HD / 16; kc_++) ldsm_x4(qa[kc_], sQ + sw(warp * 16 + (lane & 15), kc_ * 2 + (lane >> 4)));
         }
@@ -671,7 +679,9 @@ __global__ void __launch_bounds__(128, KF_PF_MINB) kf_attn_prefill_kernel(uint16
                     // cap * tanh(s / cap) = cap * (1 - 2 / (e^{2 s / cap} + 1)), brought to the log2 domain
                     if (cap2 > 0.f) v = capL * (1.f - __fdividef(2.f, exp2f(v * xb.scale * cap2) + 1.f));
                     else v *= SCB;
-                    if (dist < 0 || dist >= xb.window) v = -INFINITY;
+                    if (POOL && kt < kt0) {
+                        if ((kt - it0) * BKV + j * 8 + 2 * t4 + (e & 1) >= ((e & 2) ? nb_hi : nb_lo)) v = -INFINITY;
+                    } else if (dist < 0 || dist >= xb.window) v = -INFINITY;
                 } else if (diag) {
                     const int tcol = kt * BKV + j * 8 + 2 * t4 + (e & 1);
                     if (tcol > ((e & 2) ? p_hi : p_lo)) v = -INFINITY;
@@ -738,8 +748,12 @@ __global__ void __launch_bounds__(128, KF_PF_MINB) kf_attn_prefill_kernel(uint16
 #pragma unroll
         for (int j = 0; j < HD / 8; j++) o[j][0] *= c_lo, o[j][1] *= c_lo, o[j][2] *= c_hi, o[j][3] *= c_hi;
     }
-    const float i_lo = SIG ? xb.out_scale : (WIN ? xb.out_scale : 1.f) / l_lo, i_hi = SIG ? xb.out_scale : (WIN ? xb.out_scale : 1.f) / l_hi;
+    float i_lo = SIG ? xb.out_scale : (WIN ? xb.out_scale : 1.f) / l_lo, i_hi = SIG ? xb.out_scale : (WIN ? xb.out_scale : 1.f) / l_hi;
     const int r_lo = q0 + warp * 16 + g, r_hi = r_lo + 8, o_dim = RING ? xb.out_ld : q_dim;
+    if (POOL && xb.hgate) {
+        if (r_lo < M) i_lo *= 1.f / (1.f + expf(-xb.hgate[(size_t)r_lo * xb.ldg + h]));
+        if (r_hi < M) i_hi *= 1.f / (1.f + expf(-xb.hgate[(size_t)r_hi * xb.ldg + h]));
+    }
 #pragma unroll
     for (int j = 0; j < HD / 8; j++) {
         const int d = j * 8 + 2 * t4;
@@ -1141,6 +1155,42 @@ extern "C" int kf_attn_window_prefill(kf_ctx* ctx, void* out, int ldo, const voi
             set[ctx->device] = true;
         }
         kf_attn_prefill_kernel<64, KF_PF_BKV, 2><<<grid, 128, smem, ctx->stream>>>((uint16_t*)out, (const uint16_t*)q_bf16, kc, vc, pos_dev, M, n_head, n_kv, ring,
+                                                                                 1.f, xb);
+    }
+    KF_LAUNCH_CHECK(ctx);
+    return KF_OK;
+}
+
+// kf_attn_window_ex for a panel of M consecutive tokens of one slot on the tensor cores: kf_attn_window_prefill with mean rows of blocks of
+// `pool` positions behind the ring (pool 0: none) and a gate per head (float logits [M][ldg], NULL: none).  slot_stride covers the mean rows.
+extern "C" int kf_attn_pooled_prefill(kf_ctx* ctx, void* out, int ldo, const void* q_bf16, const void* cache, size_t slot_stride, int ring, const void* sink_bf16,
+                                      const int32_t* pos_dev, const int32_t* slot_dev, int M, int n_head, int n_kv, int hd, float scale, float softcap, int window,
+                                      int pool, const float* head_gate, int ldg, float out_scale) {
+    if (!ctx || !out || !q_bf16 || !cache || !pos_dev || !slot_dev) return KF_ERR_BAD_ARG;
+    KF_REQUIRE(ctx, (hd == 128 || hd == 64) && n_head % n_kv == 0 && M >= 1 && ring >= 1 && (window <= 0 || ring >= window) && ldo >= n_head * hd && ldo % 2 == 0,
+               "head size 64/128, GQA, ring");
+    KF_REQUIRE(ctx, pool >= 0 && (pool == 0 || window > 0), "pooled blocks lie behind a window");
+    const size_t smem = (size_t)(kPfQ + 4 * KF_PF_BKV) * hd * 2;
+    dim3 grid((M + kPfQ - 1) / kPfQ, n_head);
+    PfBias xb = {nullptr, nullptr, nullptr, ldg, slot_dev, slot_stride, 2 * n_kv * hd, scale, ring, window > 0 ? window : 0x7fffffff, softcap,
+                 (const uint16_t*)sink_bf16, ldo, out_scale, 0x7fffffff, nullptr, pool, head_gate};
+    const uint16_t* kc = (const uint16_t*)cache;
+    const uint16_t* vc = kc + (size_t)n_kv * hd;
+    if (hd == 128) {
+        static bool set[kf_ctx::kMaxDevices] = {};
+        if (!set[ctx->device]) {
+            KF_CUDA(ctx, cudaFuncSetAttribute(kf_attn_prefill_kernel<128, KF_PF_BKV, 4>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+            set[ctx->device] = true;
+        }
+        kf_attn_prefill_kernel<128, KF_PF_BKV, 4><<<grid, 128, smem, ctx->stream>>>((uint16_t*)out, (const uint16_t*)q_bf16, kc, vc, pos_dev, M, n_head, n_kv, ring,
+                                                                                  1.f, xb);
+    } else {
+        static bool set[kf_ctx::kMaxDevices] = {};
+        if (!set[ctx->device]) {
+            KF_CUDA(ctx, cudaFuncSetAttribute(kf_attn_prefill_kernel<64, KF_PF_BKV, 4>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+            set[ctx->device] = true;
+        }
+        kf_attn_prefill_kernel<64, KF_PF_BKV, 4><<<grid, 128, smem, ctx->stream>>>((uint16_t*)out, (const uint16_t*)q_bf16, kc, vc, pos_dev, M, n_head, n_kv, ring,
                                                                                  1.f, xb);
     }
     KF_LAUNCH_CHECK(ctx);

@@ -12,6 +12,8 @@
 // not grow with the sequence.  A slot is never cleared: a sequence that starts at position 0 reads only rows that it wrote.
 // One kernel serves prompts (M tokens of one slot) and decoding (one token of each of M slots): a CTA per (token, head, key split), a
 // lane per key for the scores, lanes over the value entries for the sum, online softmax per warp, warps merged at the end.
+// kf_qk_heads_prepare / kf_attn_window_ex add norms per head, mean rows of blocks that have left the window (stored behind the ring) and an
+// output gate per head.
 // Beside kf_attn_bias (attn_bias.cu: distance penalty, no rotation) and kf_attn_* (attention.cu: Qwen3's path).  No reference equivalent.
 #include <math.h>
 
@@ -112,6 +114,102 @@ __global__ void __launch_bounds__(256) kf_qk_prepare_kernel(PrepArgs a) {
     }
 }
 
+// q and k normed PER HEAD (one weight of head size for all heads of q, one for all heads of k), optionally rotated, k | v appended to the
+// ring: a warp per (token, head).  With pool_now (every token of the launch belongs to a sequence of its own) the warp of a token that
+// completes a block of `pool` positions also writes its head's part of the block's mean row.
+struct HeadsArgs {
+    float* x;  // [M][ldx]: q (H x dk) | k (G x dk) | v (G x dv), consecutive
+    uint16_t* qb;  // given: q goes there as bf16 [M][H * dk] and x keeps the projection; NULL: q replaces it in x
+    int ldx, H, G, dk, dv;
+    const uint16_t *qw, *kw;  // bf16 [dk] or NULL (not normed)
+    float eps, amp;
+    int rot_dims, layout;
+    const double* inv_freq;
+    void* cache;
+    size_t slot_stride;
+    int ring, pool, pool_now;
+    const int32_t *pos, *slot;
+};
+constexpr int HW = 4;  // warps per CTA
+template <typename TC>
+__device__ __forceinline__ float round_to(float v) { return v; }
+template <>
+__device__ __forceinline__ float round_to<uint16_t>(float v) { return bf16_bits_to_f32(f32_to_bf16_bits(v)); }
+template <typename TC>
+__device__ __forceinline__ void stc(TC* p, float v);
+template <>
+__device__ __forceinline__ void stc<uint16_t>(uint16_t* p, float v) { *p = f32_to_bf16_bits(v); }
+template <>
+__device__ __forceinline__ void stc<float>(float* p, float v) { *p = v; }
+
+template <typename TC>
+__global__ void __launch_bounds__(HW * 32) kf_qk_heads_kernel(HeadsArgs a) {
+    extern __shared__ float sm[];
+    const int m = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, u = blockIdx.y * HW + warp;
+    if (u >= a.H + 2 * a.G) return;
+    const int kind = u < a.H ? 0 : u < a.H + a.G ? 1 : 2, hh = kind == 0 ? u : kind == 1 ? u - a.H : u - a.H - a.G, n = kind == 2 ? a.dv : a.dk;
+    const int nq = a.H * a.dk, nk = a.G * a.dk, W = a.G * (a.dk + a.dv), p = a.pos[m];
+    const int col = kind == 0 ? hh * a.dk : kind == 1 ? nq + hh * a.dk : nq + nk + hh * a.dv;
+    float* src = a.x + (size_t)m * a.ldx + col;
+    float* sx  = sm + warp * max(a.dk, a.dv);
+    const uint16_t* w = kind == 0 ? a.qw : kind == 1 ? a.kw : nullptr;
+    float ss = 0.f;
+    for (int d = lane; d < n; d += 32) {
+        const float v = src[d];
+        sx[d] = v, ss = fmaf(v, v, ss);
+    }
+    float f = 1.f;
+    if (w) f = 1.0f / sqrtf(warp_sum(ss) / (float)n + a.eps);
+    const int half = a.rot_dims >> 1;
+    const bool rot = kind != 2 && half > 0;
+    if (w)
+        for (int d = lane; d < n; d += 32) sx[d] *= f * bf16_bits_to_f32(w[d]);
+    __syncwarp();
+    TC* slot_rows = (TC*)a.cache + (size_t)a.slot[m] * a.slot_stride;
+    const int coff = kind == 2 ? nk + hh * a.dv : hh * a.dk;  // this head's entries inside a cache row
+    const bool completes = kind != 0 && a.pool_now && a.pool > 0 && (p + 1) % a.pool == 0;
+    for (int d = lane; d < n; d += 32) {
+        float v = sx[d];
+        if (rot && d < a.rot_dims) {  // angle formed and reduced in double, as in kf_qk_prepare_kernel
+            const int fi = a.layout == 0 ? d >> 1 : d < half ? d : d - half, partner = a.layout == 0 ? d ^ 1 : d < half ? d + half : d - half;
+            const bool first = a.layout == 0 ? !(d & 1) : d < half;
+            const double ang = (double)p * a.inv_freq[fi];
+            float s, c;
+            sincosf((float)(ang - 6.283185307179586 * rint(ang * 0.15915494309189535)), &s, &c);
+            s *= a.amp, c *= a.amp;
+            v = first ? v * c - sx[partner] * s : v * c + sx[partner] * s;
+        }
+        if (kind == 0) {
+            if (a.qb) a.qb[(size_t)m * nq + col + d] = f32_to_bf16_bits(v);
+            else src[d] = v;
+            continue;
+        }
+        stc<TC>(slot_rows + (size_t)(p % a.ring) * W + coff + d, v);
+        if (completes) {
+            float acc = 0.f;
+            for (int j = p - a.pool + 1; j < p; j++) acc += ldc<TC>(slot_rows + (size_t)(j % a.ring) * W + coff + d);
+            acc += round_to<TC>(v);
+            stc<TC>(slot_rows + (size_t)(a.ring + p / a.pool) * W + coff + d, acc / (float)a.pool);
+        }
+    }
+}
+// the mean rows of the blocks that this launch's tokens complete (their rows are in the ring): row ring + p / pool = mean of the rows of
+// positions p - pool + 1 .. p, summed in order; a CTA per token, those that complete nothing leave at once
+template <typename TC>
+__global__ void __launch_bounds__(128) kf_kv_pool_kernel(TC* cache, size_t slot_stride, int ring, int pool, int W, const int32_t* __restrict__ pos,
+                                                         const int32_t* __restrict__ slot) {
+    const int p = pos[blockIdx.x], i = blockIdx.y * blockDim.x + threadIdx.x;
+    if ((p + 1) % pool || i >= W) return;
+    TC* rows = cache + (size_t)slot[blockIdx.x] * slot_stride;
+    float acc = 0.f;
+    int r = (p - pool + 1) % ring;
+    for (int j = 0; j < pool; j++) {
+        acc += ldc<TC>(rows + (size_t)r * W + i);
+        r = r + 1 == ring ? 0 : r + 1;
+    }
+    stc<TC>(rows + (size_t)(ring + p / pool) * W + i, acc / (float)pool);
+}
+
 struct WinArgs {
     void* out;  // [M][ldo] activation type, heads x dv
     int ldo, out_f32;
@@ -126,6 +224,11 @@ struct WinArgs {
     float scale, softcap, out_scale;
     int nsplit;  // the keys of a token are dealt to nsplit CTAs (blockIdx.z); > 1: partial (max, sum, weighted values) go to ws
     float* ws;   // [M][H][nsplit][dv + 2]
+    // pooled blocks (kf_attn_window_ex): beside the window, one key / value row for every block of `pool` positions that ends at or before
+    // p - window; block b's row sits behind the ring, at row ring + b (0: none)
+    int pool;
+    const float* hgate;  // [M][ldg] logits: head h's result is multiplied by sigmoid(hgate[m][h]) (NULL: not)
+    int ldg;
     // sigmoid-weighted attention (kf_attn_sigmoid): keys of the query's own block of `block` positions only (0: no blocks), a bias per
     // head inside the sigmoid (bf16 [H] or NULL)
     int block;
@@ -134,6 +237,7 @@ struct WinArgs {
 
 __device__ __forceinline__ void win_store(const WinArgs& a, int m, int h, int d, float o) {
     o *= a.out_scale;
+    if (a.hgate) o *= 1.f / (1.f + expf(-a.hgate[(size_t)m * a.ldg + h]));
     if (a.out_f32) ((float*)a.out)[(size_t)m * a.ldo + h * a.dv + d] = o;
     else ((uint16_t*)a.out)[(size_t)m * a.ldo + h * a.dv + d] = f32_to_bf16_bits(o);
 }
@@ -156,15 +260,22 @@ __global__ void __launch_bounds__(AW * 32) kf_attn_window_kernel(WinArgs a) {
     for (int i = 0; i < VPL; i++) acc[i] = 0.f;
     const bool vec = sizeof(TC) == 2 && a.dk % 8 == 0 && W % 8 == 0 && (a.slot_stride % 8) == 0 && (((uintptr_t)a.cache & 15) == 0);
     const float inv_cap = a.softcap > 0.f ? 1.f / a.softcap : 0.f;
-    // the visible keys are lo .. p; this CTA's share: [j_lo, j_hi), whole 32-key steps per split
-    const int lo = a.window > 0 ? max(0, p - a.window + 1) : 0, nkeys = p - lo + 1;
+    // the visible keys, numbered 0 .. nkeys - 1: nb pooled blocks, then the positions lo .. p (never more than the ring holds); this CTA's
+    // share: [j_lo, j_hi), whole 32-key steps per split
+    const int lo = a.window > 0 ? max(0, p - a.window + 1) : 0;
+    const int nb = a.pool > 0 ? max(0, p - a.window + 1) / a.pool : 0, nkeys = nb + p - lo + 1, r0 = lo % a.ring - nb;
+    auto row_of = [&](int j) -> int {  // cache row of key j
+        if (j < nb) return a.ring + j;
+        const int r = r0 + j;
+        return r >= a.ring ? r - a.ring : r;
+    };
     const int chunk = a.nsplit > 1 ? (((nkeys + a.nsplit - 1) / a.nsplit + 31) & ~31) : nkeys;
-    const int j_lo = lo + blockIdx.z * chunk, j_hi = min(p + 1, j_lo + chunk);
+    const int j_lo = blockIdx.z * chunk, j_hi = min(nkeys, j_lo + chunk);
     for (int j0 = j_lo + warp * 32; j0 < j_hi; j0 += AW * 32) {
         const int j = j0 + lane;
         float s = -INFINITY;
         if (j < j_hi) {
-            const TC* kr = base + (size_t)(j % a.ring) * W + kh * a.dk;
+            const TC* kr = base + (size_t)row_of(j) * W + kh * a.dk;
             float d0 = 0.f, d1 = 0.f;
             if (vec) {
                 for (int d = 0; d < a.dk; d += 8) {
@@ -193,7 +304,7 @@ __global__ void __launch_bounds__(AW * 32) kf_attn_window_kernel(WinArgs a) {
 #pragma unroll
             for (int e = 0; e < U; e++) {
                 pt[e] = __shfl_sync(0xffffffffu, pj, (t + e) & 31);
-                const TC* vr = base + (size_t)(min(j0 + t + e, j_hi - 1) % a.ring) * W + a.G * a.dk + kh * a.dv;
+                const TC* vr = base + (size_t)row_of(min(j0 + t + e, j_hi - 1)) * W + a.G * a.dk + kh * a.dv;
 #pragma unroll
                 for (int i = 0; i < VPL; i++) {
                     const int d = i * 32 + lane;
@@ -379,6 +490,38 @@ extern "C" int kf_qk_prepare_ex(kf_ctx* ctx, float* x, int ldx, int nq, int nk, 
     return KF_OK;
 }
 
+// x[m] = [q (H x dk) | k (G x dk) | v (G x dv)] floats at row stride ldx: every head of q and of k is RMS-normed on its own (weights bf16 [dk]
+// shared by the heads; NULL: none) and rotated (rot_dims 0: not; otherwise as kf_qk_prepare); k | v become row pos[m] % ring of the slot's
+// cache [slot][ring (+ pooled rows)][G * (dk + dv)].  q is rewritten in place, or, with q_bf16_out, goes there as bf16 [M][H * dk] instead.
+// pool > 0: whenever a token completes a block of `pool` positions (counted from 0), row ring + (block) of its slot takes the mean of the
+// block's rows as the cache holds them.  one_per_slot 1: the M tokens belong to M different slots (the means then need no launch of their own).
+extern "C" int kf_qk_heads_prepare(kf_ctx* ctx, float* x, int ldx, int H, int G, int dk, int dv, const void* q_norm_bf16, const void* k_norm_bf16, float eps, int rot_dims,
+                                   const double* inv_freq_dev, float amp, int layout, void* cache, int cache_f32, size_t slot_stride, int ring, int pool,
+                                   int one_per_slot, void* q_bf16_out, const int32_t* pos_dev, const int32_t* slot_dev, int M) {
+    if (!ctx || !x || !cache || !pos_dev || !slot_dev) return KF_ERR_BAD_ARG;
+    KF_REQUIRE(ctx, M >= 1 && H >= 1 && G >= 1 && dk >= 1 && dv >= 1 && dk <= 2048 && dv <= 2048 && ring >= 1 && ldx >= H * dk + G * (dk + dv), "shape");
+    KF_REQUIRE(ctx, rot_dims >= 0 && rot_dims <= dk && rot_dims % 2 == 0 && (rot_dims == 0 || inv_freq_dev) && (layout == 0 || layout == 1), "rotation");
+    KF_REQUIRE(ctx, pool >= 0 && (pool == 0 || ring >= pool), "the ring covers a pooled block");
+    const int W = G * (dk + dv);
+    KF_REQUIRE(ctx, slot_stride >= (size_t)ring * W, "slot stride");
+    HeadsArgs a = {};
+    a.x = x, a.qb = (uint16_t*)q_bf16_out, a.ldx = ldx, a.H = H, a.G = G, a.dk = dk, a.dv = dv, a.qw = (const uint16_t*)q_norm_bf16, a.kw = (const uint16_t*)k_norm_bf16;
+    a.eps = eps, a.amp = amp, a.rot_dims = rot_dims, a.layout = layout, a.inv_freq = inv_freq_dev, a.cache = cache, a.slot_stride = slot_stride, a.ring = ring;
+    a.pool = pool, a.pool_now = one_per_slot ? 1 : 0, a.pos = pos_dev, a.slot = slot_dev;
+    const dim3 grid(M, (H + 2 * G + HW - 1) / HW);
+    const size_t smem = (size_t)HW * std::max(dk, dv) * sizeof(float);
+    if (cache_f32) kf_qk_heads_kernel<float><<<grid, HW * 32, smem, ctx->stream>>>(a);
+    else kf_qk_heads_kernel<uint16_t><<<grid, HW * 32, smem, ctx->stream>>>(a);
+    KF_LAUNCH_CHECK(ctx);
+    if (pool > 0 && !one_per_slot) {
+        const dim3 g2(M, (W + 127) / 128);
+        if (cache_f32) kf_kv_pool_kernel<float><<<g2, 128, 0, ctx->stream>>>((float*)cache, slot_stride, ring, pool, W, pos_dev, slot_dev);
+        else kf_kv_pool_kernel<uint16_t><<<g2, 128, 0, ctx->stream>>>((uint16_t*)cache, slot_stride, ring, pool, W, pos_dev, slot_dev);
+        KF_LAUNCH_CHECK(ctx);
+    }
+    return KF_OK;
+}
+
 // out [M][ldo] (heads x dv, activation type) = attention of token m over the rows of positions max(0, pos[m] - window + 1) .. pos[m] of its
 // slot's ring (its own row appended before).  window <= 0: every position from 0; softcap <= 0: scores are not capped; sink: bf16 [H] or
 // NULL.  ring must cover the window (and, for window <= 0, every position).  max_keys_hint: an upper bound of the keys a token sees (sizes
@@ -386,15 +529,27 @@ extern "C" int kf_qk_prepare_ex(kf_ctx* ctx, float* x, int ldx, int nq, int nk, 
 extern "C" int kf_attn_window(kf_ctx* ctx, void* out, int out_f32, int ldo, const float* q, int ldq, const void* cache, int cache_f32, size_t slot_stride,
                               int ring, const void* sink_bf16, const int32_t* pos_dev, const int32_t* slot_dev, int M, int H, int G, int dk, int dv, float scale,
                               float softcap, int window, int max_keys_hint, float out_scale) {
+    return kf_attn_window_ex(ctx, out, out_f32, ldo, q, ldq, cache, cache_f32, slot_stride, ring, sink_bf16, pos_dev, slot_dev, M, H, G, dk, dv, scale, softcap, window,
+                             max_keys_hint, out_scale, 0, nullptr, 0);
+}
+// The same with pooled blocks beside the window -- pool > 0: token m also sees, for every block b of `pool` positions with
+// b * pool + pool - 1 <= pos[m] - window, the row ring + b of its slot (the mean row that kf_qk_heads_prepare writes); one softmax over all --
+// and an output gate per head: the result of head h is multiplied by sigmoid(head_gate[m * ldg + h]) (NULL: not).  max_keys_hint bounds the
+// positions (pos[m] + 1).
+extern "C" int kf_attn_window_ex(kf_ctx* ctx, void* out, int out_f32, int ldo, const float* q, int ldq, const void* cache, int cache_f32, size_t slot_stride, int ring,
+                                 const void* sink_bf16, const int32_t* pos_dev, const int32_t* slot_dev, int M, int H, int G, int dk, int dv, float scale, float softcap,
+                                 int window, int max_keys_hint, float out_scale, int pool, const float* head_gate, int ldg) {
     if (!ctx || !out || !q || !cache || !pos_dev || !slot_dev) return KF_ERR_BAD_ARG;
     KF_REQUIRE(ctx, M >= 1 && H >= 1 && G >= 1 && H % G == 0 && dk >= 1 && dv >= 1 && dv <= 512 && ring >= 1 && (window <= 0 || ring >= window),
                "value size <= 512, kv heads divide heads, the ring covers the window");
     WinArgs a = {};
     a.out = out, a.ldo = ldo, a.out_f32 = out_f32, a.q = q, a.ldq = ldq, a.cache = cache, a.slot_stride = slot_stride, a.ring = ring, a.window = window;
     a.sink = (const uint16_t*)sink_bf16, a.pos = pos_dev, a.slot = slot_dev, a.H = H, a.G = G, a.dk = dk, a.dv = dv, a.scale = scale, a.softcap = softcap, a.out_scale = out_scale;
+    KF_REQUIRE(ctx, pool >= 0 && (pool == 0 || window > 0), "pooled blocks lie behind a window");
+    a.pool = pool, a.hgate = head_gate, a.ldg = ldg;
     const size_t smem = (size_t)(dk + AW * dv + AW * 2) * sizeof(float);
     KF_REQUIRE(ctx, smem <= 48 * 1024, "key size");
-    if (window > 0) max_keys_hint = std::min(max_keys_hint, window);
+    if (window > 0) max_keys_hint = std::min(max_keys_hint, window) + (pool > 0 ? std::max(0, max_keys_hint - window) / pool : 0);
     int nsplit = 1;  // few (token, head) pairs and many keys (decoding): the keys are dealt to several CTAs so that the SMs are busy
     if (M * H < 2 * ctx->sm_count && max_keys_hint >= 4 * AW * 32)
         nsplit = std::max(1, std::min(std::min(64, (2 * ctx->sm_count) / (M * H)), max_keys_hint / (2 * AW * 32)));

@@ -68,7 +68,8 @@ __global__ void kf_depth_mix_kernel(float* __restrict__ x, float* __restrict__ h
 }
 
 // One block per (row, group).  v = x * gatefn(g) (GATE 0: none, 1: sigmoid(g + gate_bias), 2: silu(g));  r = v / sqrt(mean_group(v^2) + eps) * w;
-// GATE 3 / 4: the gate multiplies the normed result instead, r *= sigmoid(g) / silu(g).  w_shared: one weight of group size for all groups.
+// GATE 3 / 4: the gate multiplies the normed result instead, r *= sigmoid(g) / silu(g).  w_shared 1: one weight of group size for all groups;
+// 2: one number for every entry.
 // ACC: res[row] += mult * r (fp32 residual stream)  else  out[row] = r in the activation type.  w_add is added to every weight in
 // fp32 (1 for weights that are stored around zero).
 template <int GATE, bool ACC, typename TO>
@@ -98,7 +99,7 @@ __global__ void __launch_bounds__(256) kf_group_norm_kernel(TO* __restrict__ out
     ss = block_sum(ss, red);
     const float s = 1.0f / sqrtf(ss / (float)gs + eps);
     for (int i = threadIdx.x; i < gs; i += blockDim.x) {
-        float o = val(i) * s * (w_add + bf16_bits_to_f32(w[w_shared ? i : grp * gs + i]));
+        float o = val(i) * s * (w_add + bf16_bits_to_f32(w[w_shared == 2 ? 0 : w_shared ? i : grp * gs + i]));
         if (GATE == 3) o *= sigmoid_f(gr[i]);
         if (GATE == 4) {
             const float z = gr[i];
@@ -115,32 +116,114 @@ __global__ void __launch_bounds__(256) kf_group_norm_kernel(TO* __restrict__ out
     }
 }
 
-// Post-norm residual step of one row:  v = sa * a + sb * b (b optional);  res += v / sqrt(mean(v^2) + eps) * (w_add + w);  the new
-// residual row is also written in the activation type (what the next sublayer's matmul reads) when act_out is given.
-template <typename TO>
-__global__ void __launch_bounds__(256) kf_postnorm_residual_kernel(float* __restrict__ res, TO* __restrict__ act_out, const float* __restrict__ a, int lda, float sa,
-                                                                   const float* __restrict__ b, int ldb, float sb, const uint16_t* __restrict__ w, float w_add,
-                                                                   int dim, float eps) {
+// Post-norm residual step of one row:  res += mult * v / sqrt(mean(v^2) + eps) * (w_add + w)  with w per entry or (w_one) one number; v is
+//   SRC 0: sa * a + sb * b (b optional);   SRC 1: sum_j wgt[j] * y[entry_slot[j]] + shared (a token's experts; shared optional);
+//   SRC 2: a row of a bf16 table -- then the row starts the stream: res = the normed row.
+// The new residual row is also written in the activation type (what the next sublayer's matmul reads) when act is given; with `shift`
+// (rows that are one token each of different sequences) that copy is x + (prev - x) * shift, prev = the row the sequence's previous token
+// left in its tail (zeros at position 0), and the tail takes x.
+struct PostArgs {
+    float* res;
+    void* act;
+    const float *a, *b;
+    int lda, ldb;
+    float sa, sb;
+    const float *y, *wgt, *shared;
+    const int32_t* entry_slot;
+    int top;
+    const uint16_t* table;
+    const int32_t* tokens;
+    const uint16_t* w;
+    float w_add, mult;
+    int w_one, dim;
+    float eps;
+    const uint16_t* shift;
+    float* tail;
+    size_t tail_stride;
+    const int32_t *pos, *slot;
+    int cache;  // 1: dynamic shared memory holds the row of v, so its parts are read once
+};
+template <int SRC, typename TO>
+__global__ void kf_postnorm_kernel(PostArgs p) {
+    extern __shared__ float sv[];
     __shared__ float red[32];
     const int r = blockIdx.x;
-    const float* ar = a + (size_t)r * lda;
-    const float* br = b ? b + (size_t)r * ldb : nullptr;
-    auto val = [&](int i) -> float { return br ? fmaf(sb, br[i], sa * ar[i]) : sa * ar[i]; };
+    auto val = [&](int i) -> float {
+        if (SRC == 0) {
+            const float x = p.sa * p.a[(size_t)r * p.lda + i];
+            return p.b ? fmaf(p.sb, p.b[(size_t)r * p.ldb + i], x) : x;
+        }
+        if (SRC == 1) {
+            float s = 0.f;
+            for (int j = 0; j < p.top; j++) s = fmaf(p.wgt[(size_t)r * p.top + j], p.y[(size_t)p.entry_slot[(size_t)r * p.top + j] * p.dim + i], s);
+            return p.shared ? s + p.shared[(size_t)r * p.dim + i] : s;
+        }
+        return bf16_bits_to_f32(p.table[(size_t)p.tokens[r] * p.dim + i]);
+    };
     float ss = 0.f;
-    for (int i = threadIdx.x; i < dim; i += blockDim.x) {
+    for (int i = threadIdx.x; i < p.dim; i += blockDim.x) {
         const float v = val(i);
+        if (p.cache) sv[i] = v;  // read back by the same thread
         ss = fmaf(v, v, ss);
     }
     ss = block_sum(ss, red);
-    const float s = 1.0f / sqrtf(ss / (float)dim + eps);
-    for (int i = threadIdx.x; i < dim; i += blockDim.x) {
-        float* p = res + (size_t)r * dim + i;
-        const float x = *p + val(i) * s * (w_add + bf16_bits_to_f32(w[i]));
-        *p = x;
-        if (act_out) {
-            if (sizeof(TO) == 2) ((uint16_t*)act_out)[(size_t)r * dim + i] = f32_to_bf16_bits(x);
-            else ((float*)act_out)[(size_t)r * dim + i] = x;
+    const float s = 1.0f / sqrtf(ss / (float)p.dim + p.eps);
+    const float w1 = p.w_one ? p.w_add + bf16_bits_to_f32(p.w[0]) : 0.f;
+    float* tail = p.shift ? p.tail + (size_t)p.slot[r] * p.tail_stride : nullptr;
+    const bool first = p.shift && p.pos[r] == 0;
+    for (int i = threadIdx.x; i < p.dim; i += blockDim.x) {
+        float* q = p.res + (size_t)r * p.dim + i;
+        const float n = (p.cache ? sv[i] : val(i)) * s * (p.w_one ? w1 : p.w_add + bf16_bits_to_f32(p.w[i]));
+        const float x = SRC == 2 ? n : *q + p.mult * n;
+        *q = x;
+        float o = x;
+        if (p.shift) {
+            const float prev = first ? 0.f : tail[i];
+            o = fmaf(prev - x, bf16_bits_to_f32(p.shift[i]), x);
+            tail[i] = x;
         }
+        if (p.act) {
+            if (sizeof(TO) == 2) ((uint16_t*)p.act)[(size_t)r * p.dim + i] = f32_to_bf16_bits(o);
+            else ((float*)p.act)[(size_t)r * p.dim + i] = o;
+        }
+    }
+}
+template <int SRC>
+int launch_postnorm(kf_ctx* ctx, PostArgs& p, int act_f32, int rows) {
+    const size_t smem = (size_t)p.dim * sizeof(float);
+    p.cache = smem <= 32 * 1024 ? 1 : 0;
+    const int threads = rows <= 16 && p.dim >= 2048 ? 512 : 256;  // few rows: the row's loads go out side by side
+    if (act_f32) kf_postnorm_kernel<SRC, float><<<rows, threads, p.cache ? smem : 0, ctx->stream>>>(p);
+    else kf_postnorm_kernel<SRC, uint16_t><<<rows, threads, p.cache ? smem : 0, ctx->stream>>>(p);
+    KF_LAUNCH_CHECK(ctx);
+    return KF_OK;
+}
+// Token shift of a panel: out[t] = h[t] + (h[t-1] - h[t]) * w (w per entry), h[t-1] of a sequence's first row of this launch = its tail (zeros
+// at position 0); the tail then takes the sequence's last row.  The block row of t = 0 does both, so nobody else touches the tail.
+constexpr int kShiftRows = 4;
+template <typename TO>
+__global__ void kf_token_shift_kernel(TO* __restrict__ out, const float* __restrict__ h, int ldh, const uint16_t* __restrict__ w, float* __restrict__ tail,
+                                      size_t tail_stride, const int32_t* __restrict__ pos, const int32_t* __restrict__ slot, int T, int dim) {
+    const int i = blockIdx.x * blockDim.x + threadIdx.x, seq = blockIdx.z;
+    if (i >= dim) return;
+    const float wi = bf16_bits_to_f32(w[i]);
+    const int t0 = blockIdx.y * kShiftRows, t1 = min(T, t0 + kShiftRows);
+    const float* hs = h + (size_t)seq * T * ldh;
+    float prev;
+    if (t0 == 0) {
+        float* tl = tail + (size_t)slot[(size_t)seq * T] * tail_stride + i;
+        prev = *tl;
+        *tl  = hs[(size_t)(T - 1) * ldh + i];
+    } else {
+        prev = hs[(size_t)(t0 - 1) * ldh + i];
+    }
+    for (int t = t0; t < t1; t++) {
+        const float x = hs[(size_t)t * ldh + i];
+        if (pos[(size_t)seq * T + t] == 0) prev = 0.f;
+        const float o = fmaf(prev - x, wi, x);
+        if (sizeof(TO) == 2) ((uint16_t*)out)[((size_t)seq * T + t) * dim + i] = f32_to_bf16_bits(o);
+        else ((float*)out)[((size_t)seq * T + t) * dim + i] = o;
+        prev = x;
     }
 }
 
@@ -300,9 +383,43 @@ __global__ void __launch_bounds__(128) kf_moe_route_kernel(int32_t* __restrict__
         for (int j = lane; j < top; j += 32) wgt[(size_t)m * top + j] /= den;
     }
 }
-// few tokens (decode): routing and the dispatch tables in ONE block -- warps route the tokens, then thread i ranks entry i among the
-// earlier entries of its expert, the lanes of warp 0 count one expert each and scan the counts
+// The dispatch tables of a few entries by ONE block of 256 threads: entry i = (token i / top, choice i % top) goes to expert sidx[i]; thread i
+// ranks its entry among the earlier ones of its expert, the lanes of warp 0 count one expert each and scan the counts.
 constexpr int kRouteSmall = 256;
+__device__ __forceinline__ void dispatch_small(const int* sidx, int* srank, int n, int E, int top, int32_t* offsets, int32_t* entry_slot, int32_t* slot_row,
+                                               int32_t* slot_group) {
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    __syncthreads();
+    for (int i = threadIdx.x; i < n; i += blockDim.x) {
+        int r = 0;
+        for (int j = 0; j < i; j++) r += sidx[j] == sidx[i];
+        srank[i] = r;
+    }
+    __syncthreads();
+    if (warp == 0) {  // offsets: lane l counts the entries of expert e0 + l, a scan over the lanes places them behind the experts before
+        int base = 0;
+        for (int e0 = 0; e0 < E; e0 += 32) {
+            const int e = e0 + lane;
+            int c = 0;
+            for (int j = 0; j < n; j++) c += sidx[j] == e;  // e >= E matches nothing
+            int incl = c;
+#pragma unroll
+            for (int o = 1; o < 32; o <<= 1) {
+                const int up = __shfl_up_sync(0xffffffffu, incl, o);
+                if (lane >= o) incl += up;
+            }
+            if (e < E) offsets[e] = base + incl - c;
+            base += __shfl_sync(0xffffffffu, incl, 31);
+        }
+        if (lane == 0) offsets[E] = base;
+    }
+    __syncthreads();
+    for (int i = threadIdx.x; i < n; i += blockDim.x) {
+        const int e = sidx[i], sl = offsets[e] + srank[i];
+        entry_slot[i] = sl, slot_row[sl] = i / top, slot_group[sl] = e;
+    }
+}
+// few tokens (decode): routing and the dispatch tables in ONE block
 __global__ void __launch_bounds__(256) kf_moe_route_small_kernel(int32_t* __restrict__ idx, float* __restrict__ wgt, int32_t* __restrict__ offsets,
                                                                  int32_t* __restrict__ entry_slot, int32_t* __restrict__ slot_row,
                                                                  int32_t* __restrict__ slot_group, const float* __restrict__ logits, int ldl,
@@ -346,41 +463,13 @@ __global__ void __launch_bounds__(256) kf_moe_route_small_kernel(int32_t* __rest
         }
         for (int j = lane; j < top; j += 32) wgt[(size_t)m * top + j] /= den;
     }
-    __syncthreads();
-    for (int i = threadIdx.x; i < n; i += blockDim.x) {
-        int r = 0;
-        for (int j = 0; j < i; j++) r += sidx[j] == sidx[i];
-        srank[i] = r;
-    }
-    __syncthreads();
-    if (warp == 0) {  // offsets: lane l counts the entries of expert e0 + l, a scan over the lanes places them behind the experts before
-        int base = 0;
-        for (int e0 = 0; e0 < E; e0 += 32) {
-            const int e = e0 + lane;
-            int c = 0;
-            for (int j = 0; j < n; j++) c += sidx[j] == e;  // e >= E matches nothing
-            int incl = c;
-#pragma unroll
-            for (int o = 1; o < 32; o <<= 1) {
-                const int up = __shfl_up_sync(0xffffffffu, incl, o);
-                if (lane >= o) incl += up;
-            }
-            if (e < E) offsets[e] = base + incl - c;
-            base += __shfl_sync(0xffffffffu, incl, 31);
-        }
-        if (lane == 0) offsets[E] = base;
-    }
-    __syncthreads();
-    for (int i = threadIdx.x; i < n; i += blockDim.x) {
-        const int e = sidx[i], sl = offsets[e] + srank[i];
-        entry_slot[i] = sl, slot_row[sl] = i / top, slot_group[sl] = e;
-    }
+    dispatch_small(sidx, srank, n, E, top, offsets, entry_slot, slot_row, slot_group);
 }
 // one block per expert: the entries (token, choice) routed to it, ranked in entry order (ballot + popc compaction)
-__global__ void __launch_bounds__(256) kf_moe_rank_kernel(int32_t* __restrict__ rank, int32_t* __restrict__ count, const int32_t* __restrict__ idx, int n) {
+__device__ __forceinline__ void rank_expert(int32_t* rank, int32_t* count, const int32_t* idx, int n, int e) {
     __shared__ int wsum[8];
     __shared__ int base;
-    const int e = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     if (threadIdx.x == 0) base = 0;
     __syncthreads();
     for (int i0 = 0; i0 < n; i0 += 256) {
@@ -402,6 +491,9 @@ __global__ void __launch_bounds__(256) kf_moe_rank_kernel(int32_t* __restrict__ 
     }
     if (threadIdx.x == 0) count[e] = base;
 }
+__global__ void __launch_bounds__(256) kf_moe_rank_kernel(int32_t* __restrict__ rank, int32_t* __restrict__ count, const int32_t* __restrict__ idx, int n) {
+    rank_expert(rank, count, idx, n, blockIdx.x);
+}
 // offsets = exclusive scan of the counts (one thread: E is small); then each entry learns its slot
 __global__ void kf_moe_offsets_kernel(int32_t* __restrict__ offsets, const int32_t* __restrict__ count, int E) {
     if (threadIdx.x == 0 && blockIdx.x == 0) {
@@ -416,6 +508,58 @@ __global__ void kf_moe_slots_kernel(int32_t* __restrict__ entry_slot, int32_t* _
     if (i >= n) return;
     const int e = idx[i], s = offsets[e] + rank[i];
     entry_slot[i] = s, slot_row[s] = i / top, slot_group[s] = e;
+}
+// Routing from a table of token ids: row tokens[m] names the token's `top` experts, each with weight 1 / top -- no logits.  It depends on
+// the token ids alone, so ONE launch fills the tables of several layers (blockIdx.y / .x picks the layer).
+__device__ __forceinline__ int table_expert(const kf_table_route& r, int token, int j) {
+    return (int)min((unsigned)r.table[(size_t)token * r.top + j], (unsigned)(r.experts - 1));  // ids are checked when the table is loaded
+}
+__global__ void __launch_bounds__(256) kf_moe_table_small_kernel(const kf_table_route* __restrict__ routes, const int32_t* __restrict__ tokens, int M) {
+    __shared__ int sidx[kRouteSmall];
+    __shared__ int srank[kRouteSmall];
+    const kf_table_route r = routes[blockIdx.x];
+    const int n = M * r.top;
+    for (int i = threadIdx.x; i < n; i += blockDim.x) {
+        const int e = table_expert(r, tokens[i / r.top], i % r.top);
+        sidx[i] = e, r.idx[i] = e, r.wgt[i] = 1.f / (float)r.top;
+    }
+    dispatch_small(sidx, srank, n, r.experts, r.top, r.offsets, r.entry_slot, r.slot_row, r.slot_group);
+}
+__global__ void kf_moe_table_idx_kernel(const kf_table_route* __restrict__ routes, const int32_t* __restrict__ tokens, int M) {
+    const kf_table_route r = routes[blockIdx.y];
+    const int i = blockIdx.x * blockDim.x + threadIdx.x;
+    if (i < M * r.top) r.idx[i] = table_expert(r, tokens[i / r.top], i % r.top), r.wgt[i] = 1.f / (float)r.top;
+}
+__global__ void __launch_bounds__(256) kf_moe_table_rank_kernel(const kf_table_route* __restrict__ routes, int M) {
+    const kf_table_route r = routes[blockIdx.y];
+    if (blockIdx.x < r.experts) rank_expert(r.work, r.work + M * r.top, r.idx, M * r.top, blockIdx.x);
+}
+__global__ void kf_moe_table_slots_kernel(const kf_table_route* __restrict__ routes, int M) {  // offsets: every block scans the few counts itself
+    extern __shared__ int soff[];
+    const kf_table_route r = routes[blockIdx.y];
+    const int n = M * r.top, E = r.experts, lane = threadIdx.x & 31;
+    const int32_t* count = r.work + n;
+    if (threadIdx.x < 32) {
+        int base = 0;
+        for (int e0 = 0; e0 < E; e0 += 32) {
+            const int e = e0 + lane, c = e < E ? count[e] : 0;
+            int incl = c;
+#pragma unroll
+            for (int o = 1; o < 32; o <<= 1) {
+                const int up = __shfl_up_sync(0xffffffffu, incl, o);
+                if (lane >= o) incl += up;
+            }
+            if (e < E) soff[e] = base + incl - c;
+            base += __shfl_sync(0xffffffffu, incl, 31);
+        }
+    }
+    __syncthreads();
+    if (blockIdx.x == 0)
+        for (int e = threadIdx.x; e <= E; e += blockDim.x) r.offsets[e] = e < E ? soff[e] : n;
+    const int i = blockIdx.x * blockDim.x + threadIdx.x;
+    if (i >= n) return;
+    const int e = r.idx[i], sl = soff[e] + r.work[i];
+    r.entry_slot[i] = sl, r.slot_row[sl] = i / r.top, r.slot_group[sl] = e;
 }
 // out[m] = sum_j wgt[m][j] * y[slot(m, j)]  (+ sigmoid(sg[m]) * shared[m]), choices added in their routing order
 __global__ void kf_moe_combine_kernel(float* __restrict__ out, const float* __restrict__ y, const int32_t* __restrict__ entry_slot,
@@ -482,7 +626,8 @@ extern "C" int kf_depth_mix(kf_ctx* ctx, float* x, float* hist, size_t hist_stri
 
 // gate_kind 0: none; 1: x * sigmoid(gate + gate_bias); 2: x * silu(gate).  out_kind 0: bf16 bits [rows][ldo]; 1: float [rows][ldo];
 // 2: res[rows][dim] += mult * result (out is ignored).  row_idx (device, optional): source row of each output row.
-// gate_kind 3 / 4: sigmoid(gate) / silu(gate) multiply the normed result; w_shared: the weight has dim / groups entries, used by every group.
+// gate_kind 3 / 4: sigmoid(gate) / silu(gate) multiply the normed result; w_shared 1: the weight has dim / groups entries, used by every group; 2: it is one
+// number.
 // w_add: added to every weight in fp32 (1 for weights stored around zero, 0 for plain weights).  out_mult: factor on the rows written to
 // out (out_kind 0 / 1), applied in fp32 before the rounding.
 extern "C" int kf_group_rmsnorm_wadd(kf_ctx* ctx, void* out, int out_kind, int ldo, float* res, float mult, const float* x, int ldx, const float* gate, int ldg,
@@ -534,12 +679,58 @@ extern "C" int kf_group_rmsnorm(kf_ctx* ctx, void* out, int out_kind, int ldo, f
 // b may be NULL (one branch).  The norm runs over the whole row.
 extern "C" int kf_postnorm_residual(kf_ctx* ctx, float* res, void* act_out, int act_f32, const float* a, int lda, float sa, const float* b, int ldb, float sb,
                                     const void* w_bf16, float w_add, int rows, int dim, float eps) {
+    return kf_postnorm_residual_ex(ctx, res, act_out, act_f32, a, lda, sa, b, ldb, sb, w_bf16, w_add, 0, 1.f, rows, dim, eps, nullptr, nullptr, 0, nullptr, nullptr);
+}
+static bool post_common(PostArgs& p, float* res, void* act_out, const void* w_bf16, float w_add, int w_one, float mult, int dim, float eps, const void* shift_bf16,
+                        float* tail, size_t tail_stride, const int32_t* pos, const int32_t* slot) {
+    p.res = res, p.act = act_out, p.w = (const uint16_t*)w_bf16, p.w_add = w_add, p.w_one = w_one, p.mult = mult, p.dim = dim, p.eps = eps;
+    p.shift = (const uint16_t*)shift_bf16, p.tail = tail, p.tail_stride = tail_stride, p.pos = pos, p.slot = slot;
+    return !shift_bf16 || (tail && tail_stride >= (size_t)dim && pos && slot && act_out);
+}
+// The general form: the sum is multiplied by `mult`, w_one 1: the norm's weight is one number.  shift_bf16 [dim] (optional; every row then is
+// one token of a sequence of its own): act_out = x + (prev - x) * shift instead of x, prev = the sequence's tail [slot][tail_stride] (zeros at
+// position 0), which then takes x.
+extern "C" int kf_postnorm_residual_ex(kf_ctx* ctx, float* res, void* act_out, int act_f32, const float* a, int lda, float sa, const float* b, int ldb, float sb,
+                                       const void* w_bf16, float w_add, int w_one, float mult, int rows, int dim, float eps, const void* shift_bf16, float* tail,
+                                       size_t tail_stride, const int32_t* pos, const int32_t* slot) {
     if (!ctx || !res || !a || !w_bf16) return KF_ERR_BAD_ARG;
     KF_REQUIRE(ctx, rows >= 1 && dim >= 1, "shape");
-    if (act_f32)
-        kf_postnorm_residual_kernel<float><<<rows, 256, 0, ctx->stream>>>(res, (float*)act_out, a, lda, sa, b, ldb, sb, (const uint16_t*)w_bf16, w_add, dim, eps);
-    else
-        kf_postnorm_residual_kernel<uint16_t><<<rows, 256, 0, ctx->stream>>>(res, (uint16_t*)act_out, a, lda, sa, b, ldb, sb, (const uint16_t*)w_bf16, w_add, dim, eps);
+    PostArgs p = {};
+    KF_REQUIRE(ctx, post_common(p, res, act_out, w_bf16, w_add, w_one, mult, dim, eps, shift_bf16, tail, tail_stride, pos, slot), "a shift needs its tail, positions and slots");
+    p.a = a, p.lda = lda, p.sa = sa, p.b = b, p.ldb = ldb, p.sb = sb;
+    return launch_postnorm<0>(ctx, p, act_f32, rows);
+}
+// The same step over a token's experts: v = sum_j wgt[m][j] * y_slots[entry_slot[m][j]] (+ shared[m]); the combination never reaches memory.
+extern "C" int kf_experts_postnorm_residual(kf_ctx* ctx, float* res, void* act_out, int act_f32, const float* y_slots, const int32_t* entry_slot, const float* wgt,
+                                            const float* shared, int top, const void* w_bf16, float w_add, int w_one, float mult, int rows, int dim, float eps,
+                                            const void* shift_bf16, float* tail, size_t tail_stride, const int32_t* pos, const int32_t* slot) {
+    if (!ctx || !res || !y_slots || !entry_slot || !wgt || !w_bf16) return KF_ERR_BAD_ARG;
+    KF_REQUIRE(ctx, rows >= 1 && dim >= 1 && top >= 1, "shape");
+    PostArgs p = {};
+    KF_REQUIRE(ctx, post_common(p, res, act_out, w_bf16, w_add, w_one, mult, dim, eps, shift_bf16, tail, tail_stride, pos, slot), "a shift needs its tail, positions and slots");
+    p.y = y_slots, p.entry_slot = entry_slot, p.wgt = wgt, p.shared = shared, p.top = top;
+    return launch_postnorm<1>(ctx, p, act_f32, rows);
+}
+// The start of a stream: res[m] = rmsnorm(W[token[m]]) * (w_add + w); act_out and the shift as above.
+extern "C" int kf_embed_norm(kf_ctx* ctx, float* res, void* act_out, int act_f32, const kf_tensor_desc* table, const int32_t* tokens, const void* w_bf16, float w_add,
+                             int w_one, int rows, float eps, const void* shift_bf16, float* tail, size_t tail_stride, const int32_t* pos, const int32_t* slot) {
+    if (!ctx || !res || !table || !table->data_dev || !tokens || !w_bf16) return KF_ERR_BAD_ARG;
+    KF_REQUIRE(ctx, rows >= 1 && table->type == KF_T_BF16 && table->cols >= 1, "bf16 table");
+    PostArgs p = {};
+    KF_REQUIRE(ctx, post_common(p, res, act_out, w_bf16, w_add, w_one, 1.f, table->cols, eps, shift_bf16, tail, tail_stride, pos, slot), "a shift needs its tail, positions and slots");
+    p.table = (const uint16_t*)table->data_dev, p.tokens = tokens;
+    return launch_postnorm<2>(ctx, p, act_f32, rows);
+}
+// Token shift over nseq sequences of T consecutive tokens each (rows seq * T + t of h, row stride ldh): out [nseq * T][dim] in the activation
+// type = h[t] + (h[t-1] - h[t]) * w; tail [slot][tail_stride] floats hold the last row of the sequence's earlier tokens (ignored at position 0)
+// and take the last row of this step.
+extern "C" int kf_token_shift(kf_ctx* ctx, void* out, int out_f32, const float* h, int ldh, const void* w_bf16, float* tail, size_t tail_stride, const int32_t* pos,
+                              const int32_t* slot, int nseq, int T, int dim) {
+    if (!ctx || !out || !h || !w_bf16 || !tail || !pos || !slot) return KF_ERR_BAD_ARG;
+    KF_REQUIRE(ctx, nseq >= 1 && nseq <= 65535 && T >= 1 && dim >= 1 && ldh >= dim && tail_stride >= (size_t)dim, "shape");
+    dim3 grid((dim + 127) / 128, (T + kShiftRows - 1) / kShiftRows, nseq);
+    if (out_f32) kf_token_shift_kernel<float><<<grid, 128, 0, ctx->stream>>>((float*)out, h, ldh, (const uint16_t*)w_bf16, tail, tail_stride, pos, slot, T, dim);
+    else kf_token_shift_kernel<uint16_t><<<grid, 128, 0, ctx->stream>>>((uint16_t*)out, h, ldh, (const uint16_t*)w_bf16, tail, tail_stride, pos, slot, T, dim);
     KF_LAUNCH_CHECK(ctx);
     return KF_OK;
 }
@@ -628,6 +819,25 @@ extern "C" int kf_moe_route_grouped(kf_ctx* ctx, int32_t* idx, float* wgt, int32
 extern "C" int kf_moe_route(kf_ctx* ctx, int32_t* idx, float* wgt, int32_t* offsets, int32_t* entry_slot, int32_t* slot_row, int32_t* slot_group,
                             int32_t* work, const float* logits, int ldl, const void* bias_bf16, int M, int E, int top) {
     return kf_moe_route_ex(ctx, idx, wgt, offsets, entry_slot, slot_row, slot_group, work, logits, ldl, bias_bf16, M, E, top, 0);
+}
+// kf_moe_route's tables for n_routes layers at once, the experts read from tables of token ids (see kf_table_route): routes_dev is a device
+// array; max_experts / max_top bound the entries of all routes.  work of a route: M * top + experts ints.
+extern "C" int kf_moe_route_table(kf_ctx* ctx, const kf_table_route* routes_dev, int n_routes, int max_experts, int max_top, const int32_t* tokens, int M) {
+    if (!ctx || !routes_dev || !tokens) return KF_ERR_BAD_ARG;
+    KF_REQUIRE(ctx, n_routes >= 1 && n_routes <= 65535 && max_experts >= 1 && max_experts <= 8192 && max_top >= 1 && M >= 1, "shape");
+    const int n = M * max_top;
+    if (n <= kRouteSmall && (long long)max_experts * n <= 16384) {
+        kf_moe_table_small_kernel<<<n_routes, 256, 0, ctx->stream>>>(routes_dev, tokens, M);
+        KF_LAUNCH_CHECK(ctx);
+        return KF_OK;
+    }
+    kf_moe_table_idx_kernel<<<dim3((n + 255) / 256, n_routes), 256, 0, ctx->stream>>>(routes_dev, tokens, M);
+    KF_LAUNCH_CHECK(ctx);
+    kf_moe_table_rank_kernel<<<dim3(max_experts, n_routes), 256, 0, ctx->stream>>>(routes_dev, M);
+    KF_LAUNCH_CHECK(ctx);
+    kf_moe_table_slots_kernel<<<dim3((n + 255) / 256, n_routes), 256, (size_t)max_experts * sizeof(int), ctx->stream>>>(routes_dev, M);
+    KF_LAUNCH_CHECK(ctx);
+    return KF_OK;
 }
 // accumulate 1: out += the combination (the residual stream takes the experts' sum directly)
 extern "C" int kf_moe_combine_ex(kf_ctx* ctx, float* out, const float* y_slots, const int32_t* entry_slot, const float* wgt, const float* shared,

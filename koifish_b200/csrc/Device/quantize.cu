@@ -128,7 +128,10 @@ __global__ void __launch_bounds__(256) kf_f8e5m2_encode_kernel(const uint16_t* _
     }
 }
 
-extern "C" size_t kf_quant_data_bytes(int rows, int cols, int type) { return (size_t)rows * cols * kf_type_bits(type) / 8; }
+extern "C" size_t kf_quant_data_bytes(int rows, int cols, int type) {
+    if (type == KF_T_I32) return (size_t)rows * cols * 4;
+    return (size_t)rows * cols * kf_type_bits(type) / 8;
+}
 extern "C" size_t kf_quant_gama_bytes(int rows, int cols, int type, int group) {
     if (type == KF_T_NF4) return 2 * ((size_t)rows + cols + 16 * (size_t)rows);  // szGama of RT_NormalF, GeQuant.cpp:744
     if (!kf_type_packed(type) || group <= 0)

@@ -18,6 +18,7 @@ int kfType(typNUMBER t) {
         case typNUMBER::T_BINARY: return KF_T_BINARY;
         case typNUMBER::Q4_NF: return KF_T_NF4;
         case typNUMBER::Q4_AWQ: return KF_T_AWQ4;
+        case typNUMBER::I32: return KF_T_I32;
     }
     return KF_T_BF16;
 }
@@ -31,11 +32,13 @@ const char* typName(typNUMBER t) {
         case typNUMBER::T_BINARY: return "T_BINARY";
         case typNUMBER::Q4_NF: return "Q4(NF4)";
         case typNUMBER::Q4_AWQ: return "Q4(AWQ)";
+        case typNUMBER::I32: return "I32";
     }
     return "?";
 }
 double BitPE(typNUMBER t) {
     switch (t) {
+        case typNUMBER::I32: return 32;
         case typNUMBER::BF16: return 16;
         case typNUMBER::F8E5M2: return 8;
         case typNUMBER::Q4:
@@ -180,6 +183,16 @@ int GTensor::SetBF16FromDevice(const void* src) {
     int rc = Alloc(typNUMBER::BF16, 0);
     if (rc) return rc;
     return kf_d2d(ctx, data, src, szData);
+}
+bool GTensor::IdsInRange(const int32_t* ids) const {
+    for (size_t i = 0; i < size(); i++)
+        if (ids[i] < 0 || ids[i] >= id_limit) return false;
+    return true;
+}
+int GTensor::SetIdsFromHost(const int32_t* ids) {
+    int rc = Alloc(typNUMBER::I32, 0);
+    if (!rc) rc = kf_h2d(ctx, data, ids, szData);
+    return rc ? rc : kf_ctx_sync(ctx);  // the host array is the caller's
 }
 int GTensor::GetDataX(void* out) const {
     kf_tensor_desc d = Desc();

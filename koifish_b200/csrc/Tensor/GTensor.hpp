@@ -19,7 +19,8 @@ namespace koifish {
 enum class typNUMBER : uint8_t {
     BF16, F8E5M2, Q4, Q2, T_SIGN, T_BINARY,
     Q4_NF,  /* Q4 under QUANT_MODE::RTNf: NormalFloat4 + per-row LUT */
-    Q4_AWQ  /* Q4 under QUANT_MODE::AWQ: the vendor layout, stored [in_features][out_features] (GeQuant::ExTensor, GeQuant.cpp:144-200) */
+    Q4_AWQ, /* Q4 under QUANT_MODE::AWQ: the vendor layout, stored [in_features][out_features] (GeQuant::ExTensor, GeQuant.cpp:144-200) */
+    I32     /* a table of ids below id_limit (no weights) */
 };
 int kfType(typNUMBER t);               // -> KF_T_*
 const char* typName(typNUMBER t);
@@ -62,6 +63,7 @@ class GTensor : public std::enable_shared_from_this<GTensor> {
     void* data     = nullptr;  // device blob: data || gama  (GTensor.cpp:1017)
     size_t szData = 0, szGama = 0;
     int qBias = 0;
+    int id_limit = 0;  // > 0: the tensor is a table of ids 0 .. id_limit - 1 (type I32, never quantised)
     hQUANT hQuant;
     kf_ctx* ctx = nullptr;
 
@@ -80,6 +82,10 @@ class GTensor : public std::enable_shared_from_this<GTensor> {
     // szData = the qweight bytes, szGama = qzeros + scales.
     int AllocAWQ();
     size_t awqZeroBytes() const { return (size_t)(ne[1] / 128) * (ne[0] / 8) * 4; }
+    // the storage type of an un-quantised tensor, and whether host ids all lie below id_limit (kernels index with them unchecked)
+    typNUMBER plainType() const { return id_limit > 0 ? typNUMBER::I32 : typNUMBER::BF16; }
+    bool IdsInRange(const int32_t* ids) const;
+    int SetIdsFromHost(const int32_t* ids);  // type I32; the caller has checked the range
     int SetBF16FromDevice(const void* bf16_dev);  // un-quantised tensors (norms, bf16 embed)
     // GTensor::GetDataX (quantizer.cu:249-392): dequantise to a caller-provided bf16 device buffer (test hook)
     int GetDataX(void* out_bf16_dev) const;

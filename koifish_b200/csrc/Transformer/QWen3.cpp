@@ -87,7 +87,7 @@ MODEL_CARD MODEL_CARD::FromJSON(const JSON& j0) {
     if (const JSON* s = j0.path({"init", "norm_sigma"})) c.norm_sigma = (float)s->as_double(c.norm_sigma);
     std::string a = c.arch;
     std::transform(a.begin(), a.end(), a.begin(), ::toupper);
-    if (!FindArch(a)) throw std::runtime_error("model.arch '" + c.arch + "' is outside the hot path (registered: QWEN3, SIPAZEN, KIVORAX, SEDOTAR, FAZOLORN)");
+    if (!FindArch(a)) throw std::runtime_error("model.arch '" + c.arch + "' is outside the hot path (registered: QWEN3, SIPAZEN, KIVORAX, SEDOTAR, FAZOLORN, GADILIX)");
     if (const JSON* s = j0.path({"gpt", "compute_dtype"})) c.compute_f32 = s->as_string("") == "float32";
     c.logit_rows_cfg = jint(j0, {"gpt", "logit_rows"}, c.logit_rows_cfg);
     if (c.max_seq_len <= 0 || c.max_batch <= 0) throw std::runtime_error("gpt.max_seq_len / gpt.max_batch must be positive");
@@ -108,7 +108,7 @@ const ARCH_ENTRY* FindArch(const std::string& name) {
     static const ARCH_ENTRY qwen3 = {"QWEN3", nullptr, BuildQwen3, ForwardQwen3, nullptr};
     std::string a = name;
     std::transform(a.begin(), a.end(), a.begin(), ::toupper);
-    const ARCH_ENTRY* all[] = {&qwen3, SipazenArch(), KivoraxArch(), SedotarArch(), FazolornArch()};
+    const ARCH_ENTRY* all[] = {&qwen3, SipazenArch(), KivoraxArch(), SedotarArch(), FazolornArch(), GadilixArch()};
     for (const ARCH_ENTRY* e : all)
         if (a == e->name) return e;
     return nullptr;
@@ -455,7 +455,14 @@ int Fish::InitParamRandom() {
         int rg, cg, r0, c0;
         shard_window(*this, kv.first, t->ne[0], t->ne[1], &rg, &cg, &r0, &c0);
         int rc;
-        if (t->ne[0] == 1) {  // norm weights: FIX_1 (or 1 + norm_sigma*z for tests)
+        if (t->id_limit > 0) {  // a table of ids: consecutive ids from a start that differs from row to row, so a row's entries differ
+            std::vector<int32_t> ids(t->size());
+            for (int r = 0; r < t->ne[0]; r++) {
+                const uint64_t h = ((uint64_t)r + seed) * 0x9e3779b97f4a7c15ull;
+                for (int k = 0; k < t->ne[1]; k++) ids[(size_t)r * t->ne[1] + k] = (int32_t)(((h >> 33) + (uint64_t)k) % (uint64_t)t->id_limit);
+            }
+            rc = t->SetIdsFromHost(ids.data());
+        } else if (t->ne[0] == 1) {  // norm weights: FIX_1 (or 1 + norm_sigma*z for tests)
             rc = kf_fill_normal(ctx, scratch, t->size(), seed, config.norm_sigma, 1.0f);
             if (!rc) rc = t->SetBF16FromDevice(scratch);
         } else {
@@ -482,6 +489,10 @@ int Fish::SetTensor(const std::string& name, const void* host, int rows, int col
         return KF_ERR_BAD_ARG;
     }
     hGTensor t = it->second;
+    if (t->id_limit > 0) {
+        error = "tensor '" + name + "' is a table of 32-bit ids, not of weights";
+        return KF_ERR_BAD_ARG;
+    }
     int rg, cg, r0, c0;
     shard_window(*this, name, t->ne[0], t->ne[1], &rg, &cg, &r0, &c0);
     if ((rows != rg || cols != cg) && !(t->ne[0] == 1 && (size_t)rows * cols == t->size())) {
@@ -499,6 +510,28 @@ int Fish::SetTensor(const std::string& name, const void* host, int rows, int col
     kf_free(ctx, dev);
     ResetGraphs();
     if (rc) error = "SetTensor(" + name + ") -> " + kf_status_string(rc) + " : " + kf_last_error(ctx);
+    return rc;
+}
+// a table of ids (every tensor-parallel rank keeps the whole table)
+int Fish::SetTensorIds(const std::string& name, const int32_t* ids, int rows, int cols) {
+    auto it = tensors.find(name);
+    if (it == tensors.end()) {
+        error = "unknown tensor '" + name + "'";
+        return KF_ERR_BAD_ARG;
+    }
+    hGTensor t = it->second;
+    if (t->id_limit <= 0 || rows != t->ne[0] || cols != t->ne[1]) {
+        error = "tensor '" + name + "': " + (t->id_limit <= 0 ? std::string("32-bit integers cannot be a weight")
+                                                            : "expected a table [" + std::to_string(t->ne[0]) + "," + std::to_string(t->ne[1]) + "]");
+        return KF_ERR_BAD_ARG;
+    }
+    if (!t->IdsInRange(ids)) {
+        error = "tensor '" + name + "': every id must lie in 0 .. " + std::to_string(t->id_limit - 1);
+        return KF_ERR_BAD_ARG;
+    }
+    const int rc = t->SetIdsFromHost(ids);
+    ResetGraphs();
+    if (rc) error = "SetTensorIds(" + name + ") -> " + kf_status_string(rc) + " : " + kf_last_error(ctx);
     return rc;
 }
 // The window [out r0, r0 + OCl) x [in c0, c0 + ICl) of a full AWQ triple as ONE blob qweight || qzeros || scales (GTensor::AllocAWQ).  r0 and OCl
@@ -1014,7 +1047,7 @@ int Fish::LoadBlobs(const std::string& path) {
         const bool quantised = t->hQuant && t->ne[0] > 1;
         const int group      = quantised ? t->hQuant->params.T_group : 0;
         const bool type_ok   = quantised ? ((int)BitPE(tp) == t->hQuant->bits && tp != typNUMBER::BF16) || (t->hQuant->bits == 16 && tp == typNUMBER::BF16)
-                                         : tp == typNUMBER::BF16;
+                                         : tp == t->plainType();
         if (!type_ok || meta[1] != t->ne[0] || meta[2] != t->ne[1] || meta[3] != group)
             return fail("tensor '" + name + "' was saved with another shape / storage type / group than this config selects");
         if (!t->data || t->type != tp || t->szData != sz[0] || t->szGama != sz[1]) {
@@ -1028,6 +1061,7 @@ int Fish::LoadBlobs(const std::string& path) {
         if (sz[0] != t->szData || sz[1] != t->szGama) return fail("tensor '" + name + "': byte sizes do not match its shape and type");
         host.resize(t->nByte());
         if (fread(host.data(), 1, host.size(), f) != host.size()) return fail("truncated payload of '" + name + "'");
+        if (t->id_limit > 0 && !t->IdsInRange((const int32_t*)host.data())) return fail("tensor '" + name + "' holds ids out of range");
         t->qBias = meta[4];
         int rc   = kf_h2d(ctx, t->data, host.data(), host.size());
         if (!rc) rc = kf_ctx_sync(ctx);
@@ -1055,6 +1089,7 @@ static const char* kunDtype(typNUMBER t) {  // K_FLOATS, src/g_float.hpp:127-151
         case typNUMBER::Q2: return "Q<2>";
         case typNUMBER::T_SIGN: return "TERNARY";
         case typNUMBER::T_BINARY: return "BINARY";
+        case typNUMBER::I32: return "I32";
         case typNUMBER::Q4_AWQ: return nullptr;
     }
     return nullptr;
@@ -1116,7 +1151,7 @@ int Fish::LoadKun(const std::string& path, int* n_loaded, int* n_skipped) {
         }
         const hGTensor& t   = it->second;
         const bool quantised = t->hQuant && t->ne[0] > 1;
-        typNUMBER want = quantised ? t->hQuant->params.tpQuant() : typNUMBER::BF16;
+        typNUMBER want = quantised ? t->hQuant->params.tpQuant() : t->plainType();
         if (want == typNUMBER::Q4_AWQ && config.awq_repack) want = typNUMBER::Q4;  // repacked at load: stored (and saved) as the library's own Q4
         const char* dt = kunDtype(want);
         // accept the HF spelling for plain tensors ("BF16"), otherwise the K_FLOATS name this model's config selects for the tensor
@@ -1139,6 +1174,7 @@ int Fish::LoadKun(const std::string& path, int* n_loaded, int* n_skipped) {
                         std::to_string(t->szData) + " / " + std::to_string(t->szGama) + "): another group size?");
         host.resize(t->nByte());
         if (kun_read(file, e, host.data(), &err) != 0) return fail(err);
+        if (t->id_limit > 0 && !t->IdsInRange((const int32_t*)host.data())) return fail("tensor '" + e.name + "' holds ids out of range");
         t->qBias = quantised ? t->hQuant->qBias : 0;
         int rc = kf_h2d(ctx, t->data, host.data(), host.size());
         if (!rc) rc = kf_ctx_sync(ctx);

@@ -22,7 +22,8 @@ namespace koifish {
 // that mixer's sizes, and its feed-forward.  Layers of one model may differ in every size.
 struct MIXER_CARD {
     std::string type;  // "mamba2" (state-space) | "latent_attention" | "channel_delta" | "gla" | "parallel" (attention beside a gated LRU) |
-                       // "mingru" (channel-wise gated recurrence) | "attention" (sigmoid-weighted, inside blocks of positions)
+                       // "mingru" (channel-wise gated recurrence) | "attention" (Fazolorn: sigmoid-weighted, inside blocks of positions;
+                       // Gadilix: softmax over a sliding window and pooled blocks behind it)
     // state-space mixer: heads x vdim inner channels, state rows per head, B/C groups, gated-norm groups, convolution taps
     int heads = 0, vdim = 0, state = 0, groups = 1, norm_groups = 1, conv = 1;
     // latent attention: per head `dim` plain + `rot_dim` rotated query/key entries, values of vdim, latent rank; rotation on the first
@@ -49,6 +50,8 @@ struct MIXER_CARD {
     int q_rank = 0;
     // sigmoid-weighted attention: a query sees the keys of its own block of `block` consecutive positions, aligned to position 0 (0: all)
     int block = 0;
+    // beside the window of `window` positions one mean key and value for every block of `pool` positions that lies wholly before it (0: none)
+    int pool = 0;
     // channel-wise gated recurrence (minGRU): channels of the state
     int width = 0;
     // two mixers side by side that read the same input (Sedotar's "parallel"): this card is the left one, `right` the other; the result is
@@ -67,10 +70,12 @@ struct MOE_CARD {
     bool sigmoid_route = false;
     int groups = 1, keep = 1;
     float route_scale = 1.f;
+    bool table_route = false;  // no router: a table [vocab][top] names the experts of every token id, each with weight 1 / top
 };
 struct LAYER_CARD {
     MIXER_CARD mixer;
     MOE_CARD mlp;
+    int owner = -1;  // the layer whose tensors this layer runs on (-1: its own)
 };
 
 struct MODEL_CARD {
@@ -215,6 +220,7 @@ const ARCH_ENTRY* SipazenArch();  // Sipazen.cpp
 const ARCH_ENTRY* KivoraxArch();  // Kivorax.cpp
 const ARCH_ENTRY* SedotarArch();  // Sedotar.cpp
 const ARCH_ENTRY* FazolornArch(); // Fazolorn.cpp
+const ARCH_ENTRY* GadilixArch();  // Gadilix.cpp
 
 // ---- the model ------------------------------------------------------------------------------------------------------------
 struct Fish {
@@ -279,6 +285,7 @@ struct Fish {
     int Build();                 // allocate tensors + buffers (Fish::MakeInstance -> Build, Fish.cpp:13-95)
     int InitParamRandom();       // huTensor::InitParam random path + quantise at load
     int SetTensor(const std::string& hf_name, const void* host_bf16, int rows, int cols);  // SERIALIZE path: full (unsharded) tensor
+    int SetTensorIds(const std::string& hf_name, const int32_t* ids, int rows, int cols);  // a table of 32-bit ids
     // vendor AWQ arrays of one linear (full shape), cut to this rank's window and kept in the vendor layout (GeQuant::ExTensor, GeQuant.cpp:144-200)
     int SetTensorAWQ(const std::string& hf_name, const void* qweight_i32, const void* qzeros_i32, const void* scales_f16, int in_features, int out_features);
     bool all_resident = false;  // every tensor has device data (checked once by Forward)

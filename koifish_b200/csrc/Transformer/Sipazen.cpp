@@ -359,27 +359,36 @@ int LatentAttention::cuInfer(int M, const float* u, int ldu, int off_q, int off_
     return KF_OK;
 }
 
-int MoE::cuInfer(int M, const float* u, int ldu, int off_router, int off_sg, float* into_residual) {
+int MoE::Experts(int M, const int32_t* offsets, const int32_t* slot_row, const int32_t* slot_group) {
     Fish& f = *hFish;
     std::string* hFishErr = &f.error;
     HybridScratch& s = *f.hscratch;
     const int E = f.config.n_embd, X = card.experts, top = card.top;
     const int ak = f.config.compute_f32 ? 1 : 0;
+    const void* const* tb = (const void* const*)tables;
+    KF_TRY(kf_linear_grouped(f.ctx, s.h1, card.ff, tb, tb + X, X, card.ff, E, s.hact, ak, E, offsets, slot_group, slot_row, M * top));
+    KF_TRY(kf_linear_grouped(f.ctx, s.yslots, E, tb + 2 * X, nullptr, X, E, card.ff, s.h1, ak, card.ff, offsets, slot_group, nullptr, M * top));
+    if (card.shared_ff > 0) {
+        kf_tensor_desc dg = sh_gate->Desc(), du = sh_up->Desc();
+        KF_TRY(kf_linear_g_swiglu(f.ctx, s.hs, card.shared_ff, &dg, &du, s.hact, ak, E, M));
+        KF_TRY(Lin(f, s.shared, sh_down, s.hs, M));
+    }
+    return KF_OK;
+}
+
+int MoE::cuInfer(int M, const float* u, int ldu, int off_router, int off_sg, float* into_residual) {
+    Fish& f = *hFish;
+    std::string* hFishErr = &f.error;
+    HybridScratch& s = *f.hscratch;
+    const int E = f.config.n_embd, X = card.experts, top = card.top;
     const void* rb = router_b ? router_b->data : nullptr;
     if (card.sigmoid_route)
         KF_TRY(kf_moe_route_grouped(f.ctx, s.idx, s.wgt, s.offsets, s.entry_slot, s.slot_row, s.slot_group, s.work, u + off_router, ldu, rb, M, X, top, card.groups,
                                     card.keep, card.route_scale));
     else
         KF_TRY(kf_moe_route(f.ctx, s.idx, s.wgt, s.offsets, s.entry_slot, s.slot_row, s.slot_group, s.work, u + off_router, ldu, rb, M, X, top));
-    const void* const* tb = (const void* const*)tables;
-    KF_TRY(kf_linear_grouped(f.ctx, s.h1, card.ff, tb, tb + X, X, card.ff, E, s.hact, ak, E, s.offsets, s.slot_group, s.slot_row, M * top));
-    KF_TRY(kf_linear_grouped(f.ctx, s.yslots, E, tb + 2 * X, nullptr, X, E, card.ff, s.h1, ak, card.ff, s.offsets, s.slot_group, nullptr, M * top));
+    KF_TRY(Experts(M, s.offsets, s.slot_row, s.slot_group));
     const bool sh = card.shared_ff > 0;
-    if (sh) {
-        kf_tensor_desc dg = sh_gate->Desc(), du = sh_up->Desc();
-        KF_TRY(kf_linear_g_swiglu(f.ctx, s.hs, card.shared_ff, &dg, &du, s.hact, ak, E, M));
-        KF_TRY(Lin(f, s.shared, sh_down, s.hs, M));
-    }
     KF_TRY(kf_moe_combine_ex(f.ctx, into_residual ? into_residual : s.sub, s.yslots, s.entry_slot, s.wgt, sh ? s.shared : nullptr, sh ? u + off_sg : nullptr, ldu,
                              M, E, top, into_residual ? 1 : 0));
     return KF_OK;

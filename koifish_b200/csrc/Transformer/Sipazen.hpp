@@ -69,8 +69,12 @@ struct MoE : GeNeuron {
     hGTensor router, router_b;  // router_b: bias of the softmax routing, or the selection correction of the sigmoid routing
     std::vector<hGTensor> gate, up, down;
     hGTensor sh_gate, sh_up, sh_down, sh_sg;
+    hGTensor table;           // experts by token id (card.table_route): then `route` below replaces the router and the scratch's dispatch tables
+    kf_table_route route = {};
     void** tables = nullptr;  // device: [3][experts] weight pointers (gate | up | down)
     int Prepare();
+    // the chosen experts of every token (-> yslots) and the shared expert (-> shared) on the normed input in hact, once the dispatch tables stand
+    int Experts(int M, const int32_t* offsets, const int32_t* slot_row, const int32_t* slot_group);
     // into_residual: the weighted sum of the experts is added to that buffer instead of being written to the sublayer result
     int cuInfer(int M, const float* u, int ldu, int off_router, int off_sg, float* into_residual = nullptr);
 };

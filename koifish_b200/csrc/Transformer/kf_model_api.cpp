@@ -97,6 +97,15 @@ extern "C" int kf_model_set_tensor(kf_model* m, const char* name, const void* ho
         return KF_ERR_BAD_ARG;
     }
 }
+extern "C" int kf_model_set_tensor_i32(kf_model* m, const char* name, const int32_t* host, int rows, int cols) {
+    if (!m || !name || !host) return KF_ERR_BAD_ARG;
+    try {
+        return m->fish->SetTensorIds(name, host, rows, cols);
+    } catch (const std::exception& e) {
+        m->fish->error = e.what();
+        return KF_ERR_BAD_ARG;
+    }
+}
 extern "C" int kf_model_set_tensor_awq(kf_model* m, const char* name, const void* qweight, const void* qzeros, const void* scales, int in_features,
                                        int out_features) {
     if (!m || !name) return KF_ERR_BAD_ARG;
@@ -531,14 +540,22 @@ extern "C" int kf_model_load_safetensors(kf_model* m, const char* path_or_dir, i
                     skipped++;
                     continue;
                 }
-                if (e.dtype != "BF16" && e.dtype != "F16" && e.dtype != "F32") throw std::runtime_error("'" + e.name + "': dtype " + e.dtype + " cannot be a weight");
-                if (e.shape.empty() || e.shape.size() > 3) throw std::runtime_error("'" + e.name + "': expected a vector, a matrix or a stack of matrices");
-                int64_t rows = 1;  // a stack of matrices [n][r][c] is held as [n * r][c]
+                const bool ids = m->fish->GetTensor(e.name)->id_limit > 0;
+                if (ids && e.dtype != "I32") throw std::runtime_error("'" + e.name + "': a table of ids is stored as I32, found " + e.dtype);
+                if (!ids && e.dtype != "BF16" && e.dtype != "F16" && e.dtype != "F32") throw std::runtime_error("'" + e.name + "': dtype " + e.dtype + " cannot be a weight");
+                if (e.shape.size() > 3) throw std::runtime_error("'" + e.name + "': expected a number, a vector, a matrix or a stack of matrices");
+                int64_t rows = 1;  // a stack of matrices [n][r][c] is held as [n * r][c], a single number (shape []) as [1][1]
                 for (size_t d = 0; d + 1 < e.shape.size(); d++) rows *= e.shape[d];
-                const int64_t cols = e.shape.back();
+                const int64_t cols = e.shape.empty() ? 1 : e.shape.back();
                 if (rows <= 0 || cols <= 0 || rows > 0x7fffffff || cols > 0x7fffffff) throw std::runtime_error("'" + e.name + "': bad shape");
                 raw.resize(e.end - e.begin);
                 if (kf_st_read(f, e, raw.data(), &err) != 0) throw std::runtime_error(err);
+                if (ids) {
+                    const int rci = m->fish->SetTensorIds(e.name, (const int32_t*)raw.data(), (int)rows, (int)cols);
+                    if (rci) return rci;
+                    loaded++;
+                    continue;
+                }
                 bf.resize((size_t)rows * cols);
                 kf_st_to_bf16(e.dtype, raw.data(), bf.size(), bf.data());
                 const int rc = m->fish->SetTensor(e.name, bf.data(), (int)rows, (int)cols);
