@@ -71,15 +71,15 @@ def attention(z, m, W, p, eps):
     k = rmsnorm(lin(W, p + "k", z).view(T, G, dk), W[p + "k.norm"], eps)
     v = lin(W, p + "v", z).view(T, G, dv)
     gate = torch.sigmoid(lin(W, p + "g", z))  # [T, H]
+    kv_of = [h // (H // G) for h in range(H)]  # the kv head of every query head
+    means = [(k[b * P:(b + 1) * P].mean(0), v[b * P:(b + 1) * P].mean(0)) for b in range(T // P)] if P else []
     out = torch.zeros(T, H, dv, dtype=D)
     for i in range(T):
         blocks, toks = visible(i, S, P)
-        keys = torch.stack([k[b * P:(b + 1) * P].mean(0) for b in blocks] + [k[j] for j in toks])
-        vals = torch.stack([v[b * P:(b + 1) * P].mean(0) for b in blocks] + [v[j] for j in toks])
-        for h in range(H):
-            g = h // (H // G)
-            w = torch.softmax((keys[:, g] @ q[i, h]) * scale, 0)
-            out[i, h] = gate[i, h] * (w @ vals[:, g])
+        keys = torch.stack([means[b][0] for b in blocks] + [k[j] for j in toks])[:, kv_of]  # [n, H, dk]
+        vals = torch.stack([means[b][1] for b in blocks] + [v[j] for j in toks])[:, kv_of]
+        w = torch.softmax((keys * q[i]).sum(-1) * scale, 0)  # [n, H]
+        out[i] = gate[i][:, None] * (w[:, :, None] * vals).sum(0)
     return lin(W, p + "o", out.reshape(T, H * dv))
 
 

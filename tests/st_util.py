@@ -12,8 +12,9 @@ def write_safetensors(path, tensors, metadata=None):
     if metadata:
         header["__metadata__"] = metadata
     for name, dt, a in tensors:
+        shape = list(np.shape(a))  # [] for a single number
         a = np.ascontiguousarray(a, dtype=DT[dt])
-        header[name] = {"dtype": dt, "shape": list(a.shape), "data_offsets": [off, off + a.nbytes]}
+        header[name] = {"dtype": dt, "shape": shape, "data_offsets": [off, off + a.nbytes]}
         blobs.append(a.tobytes())
         off += a.nbytes
     text = json.dumps(header, separators=(",", ":")).encode()
