@@ -1,9 +1,10 @@
-"""Prefill and decode throughput of a hybrid stack (bench.py --compare-arch sipazen | kivorax | sedotar | fazolorn) beside the closest existing
+"""Prefill and decode throughput of a hybrid stack (bench.py --compare-arch sipazen | kivorax | sedotar | fazolorn | gadilix) beside the closest existing
 models at equal width, depth and active feed-forward width: Sipazen beside Qwen3; Kivorax beside Sipazen (the other recurrence + attention +
 experts stack of this runtime) and Qwen3; Sedotar (sliding-window attention beside a delta rule, dense feed-forward) beside Kivorax with
 dense feed-forwards (delta-rule layers and attention layers alternating) and Qwen3; Fazolorn (minGRU, sigmoid block attention and latent
-attention layers with routed experts) beside Sipazen (state-space and latent attention layers with routed experts) and Qwen3.  All bf16
-with random weights.  One JSON line per (model, size).
+attention layers with routed experts) beside Sipazen (state-space and latent attention layers with routed experts) and Qwen3; Gadilix
+(windowed attention beside pooled blocks, experts by token id beside a shared one) beside Sipazen (the same experts and shared expert behind a
+router), Sedotar (the same attention heads and window, dense feed-forward) and Qwen3.  All bf16 with random weights.  One JSON line per (model, size).
 
     prefill: a prompt of --prompt tokens through the model's own step function in panels, timed with CUDA events after 3 warm-up prompts
     decode : the device-resident greedy loop (one CUDA-graph replay per token) at context --prompt, after W warm-up tokens
@@ -101,6 +102,16 @@ def fazolorn_config(p):
             "loop": {"start": 0, "stop": len(layers), "times": 1}, "layers": layers}
 
 
+def gadilix_config(p):
+    """as many layers as the preset's pattern, each attention (head size 128, 4 query heads per kv head, the preset's window, blocks of 16
+    positions behind it) and the preset's experts, top and shared expert, chosen by token id"""
+    w, d, m = p["width"], p["sdt"], p["moe"]
+    ly = {"type": "attention",
+          "mixer": dict(heads=d["heads"], kv_heads=d["kv_heads"], dim=128, vdim=128, scale=128 ** -0.5, mask=dict(size=d["window"], pool=16)),
+          "mlp": {"kind": "moe", "router": {"experts": m["experts"], "top": m["top"]}, "expert": {"ff": m["ff"]}, "shared": {"ff": m["shared"]}}}
+    return {"architecture": "Gadilix", "vocab": p["vocab"], "width": w, "residual_mult": 0.5, "norm": {"eps": 1e-5}, "layers": [ly] * len(p["pattern"])}
+
+
 def kivorax_dense_config(p):
     """Kivorax at the size of sedotar_config: delta-rule layers and attention (+ LRU) layers alternating, a dense feed-forward of the same
     width in every layer, no side input"""
@@ -156,6 +167,9 @@ def run(args, ctx, stream):
                                "init": {"sigma": 0.02, "norm_sigma": 0.02}}
         if args.compare_arch == "fazolorn":
             cfgs["fazolorn"] = {"hf_config": fazolorn_config(p), "gpt": dict(gpt), "init": {"sigma": 0.02, "norm_sigma": 0.02}}
+        if args.compare_arch == "gadilix":
+            cfgs["gadilix"] = {"hf_config": gadilix_config(p), "gpt": dict(gpt), "init": {"sigma": 0.02, "norm_sigma": 0.02}}
+            cfgs["sedotar"] = {"hf_config": sedotar_config(p), "gpt": dict(gpt), "init": {"sigma": 0.02, "norm_sigma": 0.02}}
         if args.compare_arch != "sedotar":
             cfgs["sipazen"] = {"hf_config": sipazen_config(p), "gpt": {"max_seq_len": P + args.steps + args.warmup + 64, "max_batch": 1, "max_prefill": panel},
                                "init": {"sigma": 0.02, "norm_sigma": 0.02}}
