@@ -612,10 +612,19 @@ __global__ void __launch_bounds__(128, KF_PF_MINB) kf_attn_prefill_kernel(uint16
         cp16(sQ + sw(r, c), q + (size_t)(ok ? q0 + r : 0) * q_dim + (size_t)h * HD + c * 8, ok);
     }
     auto load_kv = [&](int kt, int buf) {
+        const int tb = RING ? max(kt, 0) * BKV % xb.ring : 0;
         for (int i = tid; i < BKV * CH; i += 128) {
             const int r = i / CH, c = i % CH;
             // rows past kv_len are masked below; keep the address inside the cache (WIN: any row of the ring will do for those)
-            const int t = (POOL && kt < kt0) ? xb.ring + min((kt - it0) * BKV + r, nb_max - 1) : RING ? (kt * BKV + r) % xb.ring : min(kt * BKV + r, max_seq - 1);
+            int t;
+            if (POOL && kt < kt0) {
+                t = xb.ring + min((kt - it0) * BKV + r, nb_max - 1);
+            } else if (RING) {
+                t = tb + r;
+                if (t >= xb.ring) t = xb.ring >= BKV ? t - xb.ring : t % xb.ring;
+            } else {
+                t = min(kt * BKV + r, max_seq - 1);
+            }
             cp16(sK + buf * (BKV * HD * 2) + sw(r, c), kc + (size_t)t * kv_dim + (size_t)kvh * HD + c * 8, true);
             cp16(sV + buf * (BKV * HD * 2) + sw(r, c), vc + (size_t)t * kv_dim + (size_t)kvh * HD + c * 8, true);
         }
@@ -629,7 +638,6 @@ __global__ void __launch_bounds__(128, KF_PF_MINB) kf_attn_prefill_kernel(uint16
     for (int j = 0; j < HD / 8; j++) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
     float m_lo = -INFINITY, m_hi = -INFINITY, l_lo = 0.f, l_hi = 0.f;
     const int p_lo = pos0 + q0 + warp * 16 + g, p_hi = p_lo + 8;  // positions of this thread's two query rows
-    const int nb_lo = (POOL && xb.pool > 0) ? max(0, p_lo - xb.window + 1) / xb.pool : 0, nb_hi = (POOL && xb.pool > 0) ? max(0, p_hi - xb.window + 1) / xb.pool : 0;
     // softmax((q.k)/sqrt(hd)) = 2^((q.k - max) * log2(e)/sqrt(hd)) / sum ; BIAS: the scores are brought to the log2 domain where the penalty joins
     const float SC = ROWS ? 1.f : 1.4426950408889634f / sqrt_hd, SCB = xb.scale * 1.4426950408889634f;
     const float cap2 = (WIN && xb.softcap > 0.f) ? 2.f * 1.4426950408889634f / xb.softcap : 0.f, capL = xb.softcap * 1.4426950408889634f;
@@ -662,6 +670,20 @@ __global__ void __launch_bounds__(128, KF_PF_MINB) kf_attn_prefill_kernel(uint16
         // ---- scale, causal mask, online softmax (rows g and g + 8 of the warp's 16) ----
         float mx_lo = -INFINITY, mx_hi = -INFINITY;
         const bool diag = (kt + 1) * BKV > pos0 + q0;  // only tiles that reach the panel can contain masked columns
+        // WIN: the columns of this tile that the two rows see, relative to this thread's first one: a run [lo, hi] per row; tiles that all 64
+        // queries see whole need no mask
+        bool wmask = false;
+        int w_lo = 0, w_hi = 0, x_lo = 0, x_hi = 0;
+        if (WIN) {
+            if (POOL && kt < kt0) {
+                const int c0 = (kt - it0) * BKV + 2 * t4;
+                wmask = true, w_lo = x_lo = -BKV;
+                w_hi = max(0, p_lo - xb.window + 1) / xb.pool - 1 - c0, x_hi = max(0, p_hi - xb.window + 1) / xb.pool - 1 - c0;
+            } else {
+                wmask = diag || kt * BKV <= pos0 + q0 + kPfQ - 1 - xb.window;
+                w_hi = p_lo - kt * BKV - 2 * t4, x_hi = w_hi + 8, w_lo = w_hi - xb.window + 1, x_lo = w_lo + 8;
+            }
+        }
 #pragma unroll
         for (int j = 0; j < BKV / 8; j++) {
 #pragma unroll
@@ -675,13 +697,11 @@ __global__ void __launch_bounds__(128, KF_PF_MINB) kf_attn_prefill_kernel(uint16
                     const int tcol = kt * BKV + j * 8 + 2 * t4 + (e & 1);
                     v = (tcol > ((e & 2) ? p_hi : p_lo) || tcol < ((e & 2) ? b_hi : b_lo)) ? 0.f : __fdividef(1.f, 1.f + exp2f(-fmaf(v, SCB, hb2)));
                 } else if (WIN) {
-                    const int dist = ((e & 2) ? p_hi : p_lo) - (kt * BKV + j * 8 + 2 * t4 + (e & 1));
                     // cap * tanh(s / cap) = cap * (1 - 2 / (e^{2 s / cap} + 1)), brought to the log2 domain
                     if (cap2 > 0.f) v = capL * (1.f - __fdividef(2.f, exp2f(v * xb.scale * cap2) + 1.f));
                     else v *= SCB;
-                    if (POOL && kt < kt0) {
-                        if ((kt - it0) * BKV + j * 8 + 2 * t4 + (e & 1) >= ((e & 2) ? nb_hi : nb_lo)) v = -INFINITY;
-                    } else if (dist < 0 || dist >= xb.window) v = -INFINITY;
+                    const int col = j * 8 + (e & 1);
+                    if (wmask && ((e & 2) ? (col > x_hi || col < x_lo) : (col > w_hi || col < w_lo))) v = -INFINITY;
                 } else if (diag) {
                     const int tcol = kt * BKV + j * 8 + 2 * t4 + (e & 1);
                     if (tcol > ((e & 2) ? p_hi : p_lo)) v = -INFINITY;
@@ -1136,7 +1156,7 @@ extern "C" int kf_attn_window_prefill(kf_ctx* ctx, void* out, int ldo, const voi
                "head size 64/128, GQA, ring");
     const size_t smem = (size_t)(kPfQ + 4 * KF_PF_BKV) * hd * 2;
     dim3 grid((M + kPfQ - 1) / kPfQ, n_head);
-    PfBias xb = {nullptr, nullptr, nullptr, 0, slot_dev, slot_stride, 2 * n_kv * hd, scale, ring, window > 0 ? window : 0x7fffffff, softcap,
+    PfBias xb = {nullptr, nullptr, nullptr, 0, slot_dev, slot_stride, 2 * n_kv * hd, scale, ring, window > 0 ? window : 0x3fffffff, softcap,
                  (const uint16_t*)sink_bf16, ldo, out_scale};
     const uint16_t* kc = (const uint16_t*)cache;
     const uint16_t* vc = kc + (size_t)n_kv * hd;
@@ -1172,7 +1192,7 @@ extern "C" int kf_attn_pooled_prefill(kf_ctx* ctx, void* out, int ldo, const voi
     KF_REQUIRE(ctx, pool >= 0 && (pool == 0 || window > 0), "pooled blocks lie behind a window");
     const size_t smem = (size_t)(kPfQ + 4 * KF_PF_BKV) * hd * 2;
     dim3 grid((M + kPfQ - 1) / kPfQ, n_head);
-    PfBias xb = {nullptr, nullptr, nullptr, ldg, slot_dev, slot_stride, 2 * n_kv * hd, scale, ring, window > 0 ? window : 0x7fffffff, softcap,
+    PfBias xb = {nullptr, nullptr, nullptr, ldg, slot_dev, slot_stride, 2 * n_kv * hd, scale, ring, window > 0 ? window : 0x3fffffff, softcap,
                  (const uint16_t*)sink_bf16, ldo, out_scale, 0x7fffffff, nullptr, pool, head_gate};
     const uint16_t* kc = (const uint16_t*)cache;
     const uint16_t* vc = kc + (size_t)n_kv * hd;

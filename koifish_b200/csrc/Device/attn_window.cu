@@ -47,7 +47,7 @@ struct PrepArgs {
 
 template <typename TC>
 __global__ void __launch_bounds__(256) kf_qk_prepare_kernel(PrepArgs a) {
-    extern __shared__ float sm[];
+    extern __shared__ __align__(16) float sm[];
     __shared__ float red[32];
     const int m = blockIdx.x, n = a.nq + a.nk, half = a.rot_dims >> 1;
     float* sx = sm;          // [nq + nk] normed, not yet rotated
@@ -144,7 +144,7 @@ __device__ __forceinline__ void stc<float>(float* p, float v) { *p = v; }
 
 template <typename TC>
 __global__ void __launch_bounds__(HW * 32) kf_qk_heads_kernel(HeadsArgs a) {
-    extern __shared__ float sm[];
+    extern __shared__ __align__(16) float sm[];
     const int m = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, u = blockIdx.y * HW + warp;
     if (u >= a.H + 2 * a.G) return;
     const int kind = u < a.H ? 0 : u < a.H + a.G ? 1 : 2, hh = kind == 0 ? u : kind == 1 ? u - a.H : u - a.H - a.G, n = kind == 2 ? a.dv : a.dk;
@@ -245,7 +245,7 @@ __device__ __forceinline__ void win_store(const WinArgs& a, int m, int h, int d,
 constexpr int AW = 4;  // warps per CTA
 template <typename TC, int VPL>
 __global__ void __launch_bounds__(AW * 32) kf_attn_window_kernel(WinArgs a) {
-    extern __shared__ float sm[];
+    extern __shared__ __align__(16) float sm[];
     float* sq   = sm;                // [dk]
     float* sacc = sq + a.dk;         // [AW][dv]
     float* sml  = sacc + AW * a.dv;  // [AW][2]
@@ -259,6 +259,9 @@ __global__ void __launch_bounds__(AW * 32) kf_attn_window_kernel(WinArgs a) {
 #pragma unroll
     for (int i = 0; i < VPL; i++) acc[i] = 0.f;
     const bool vec = sizeof(TC) == 2 && a.dk % 8 == 0 && W % 8 == 0 && (a.slot_stride % 8) == 0 && (((uintptr_t)a.cache & 15) == 0);
+    // a lane's value entries: VPL consecutive ones (one load per key) when they fill the head exactly and are aligned, else every 32nd
+    const bool run = sizeof(TC) == 2 && a.dv == 32 * VPL && (VPL == 2 || VPL == 4) && vec && (a.G * a.dk) % 8 == 0;
+    auto d_of = [&](int i) { return run ? lane * VPL + i : i * 32 + lane; };
     const float inv_cap = a.softcap > 0.f ? 1.f / a.softcap : 0.f;
     // the visible keys, numbered 0 .. nkeys - 1: nb pooled blocks, then the positions lo .. p (never more than the ring holds); this CTA's
     // share: [j_lo, j_hi), whole 32-key steps per split
@@ -278,12 +281,14 @@ __global__ void __launch_bounds__(AW * 32) kf_attn_window_kernel(WinArgs a) {
             const TC* kr = base + (size_t)row_of(j) * W + kh * a.dk;
             float d0 = 0.f, d1 = 0.f;
             if (vec) {
+#pragma unroll 4
                 for (int d = 0; d < a.dk; d += 8) {
                     const uint4 kv = *reinterpret_cast<const uint4*>((const uint16_t*)kr + d);
-                    d0 = fmaf(bf16lo(kv.x), sq[d], d0), d1 = fmaf(bf16hi(kv.x), sq[d + 1], d1);
-                    d0 = fmaf(bf16lo(kv.y), sq[d + 2], d0), d1 = fmaf(bf16hi(kv.y), sq[d + 3], d1);
-                    d0 = fmaf(bf16lo(kv.z), sq[d + 4], d0), d1 = fmaf(bf16hi(kv.z), sq[d + 5], d1);
-                    d0 = fmaf(bf16lo(kv.w), sq[d + 6], d0), d1 = fmaf(bf16hi(kv.w), sq[d + 7], d1);
+                    const float4 qa = *reinterpret_cast<const float4*>(sq + d), qb = *reinterpret_cast<const float4*>(sq + d + 4);
+                    d0 = fmaf(bf16lo(kv.x), qa.x, d0), d1 = fmaf(bf16hi(kv.x), qa.y, d1);
+                    d0 = fmaf(bf16lo(kv.y), qa.z, d0), d1 = fmaf(bf16hi(kv.y), qa.w, d1);
+                    d0 = fmaf(bf16lo(kv.z), qb.x, d0), d1 = fmaf(bf16hi(kv.z), qb.y, d1);
+                    d0 = fmaf(bf16lo(kv.w), qb.z, d0), d1 = fmaf(bf16hi(kv.w), qb.w, d1);
                 }
             } else {
                 for (int d = 0; d < a.dk; d++) d0 = fmaf(ldc<TC>(kr + d), sq[d], d0);
@@ -298,17 +303,28 @@ __global__ void __launch_bounds__(AW * 32) kf_attn_window_kernel(WinArgs a) {
         for (int i = 0; i < VPL; i++) acc[i] *= corr;
         mx = nm;
         const int nk = min(32, j_hi - j0);
-        constexpr int U = VPL <= 4 ? 4 : (VPL <= 8 ? 2 : 1);  // keys per step: their value loads are issued together
+        constexpr int U = VPL <= 4 ? 8 : (VPL <= 8 ? 2 : 1);  // keys per step: their value loads are issued together
         for (int t = 0; t < nk; t += U) {
             float pt[U], x[U][VPL];
 #pragma unroll
             for (int e = 0; e < U; e++) {
                 pt[e] = __shfl_sync(0xffffffffu, pj, (t + e) & 31);
                 const TC* vr = base + (size_t)row_of(min(j0 + t + e, j_hi - 1)) * W + a.G * a.dk + kh * a.dv;
+                if (run) {
+                    const uint16_t* vp = (const uint16_t*)vr + lane * VPL;
+                    if (VPL == 4) {
+                        const uint2 pk = *reinterpret_cast<const uint2*>(vp);
+                        x[e][0] = bf16lo(pk.x), x[e][1] = bf16hi(pk.x), x[e][2 % VPL] = bf16lo(pk.y), x[e][3 % VPL] = bf16hi(pk.y);
+                    } else {
+                        const uint32_t pk = *reinterpret_cast<const uint32_t*>(vp);
+                        x[e][0] = bf16lo(pk), x[e][1] = bf16hi(pk);
+                    }
+                } else {
 #pragma unroll
-                for (int i = 0; i < VPL; i++) {
-                    const int d = i * 32 + lane;
-                    x[e][i] = d < a.dv ? ldc<TC>(vr + d) : 0.f;
+                    for (int i = 0; i < VPL; i++) {
+                        const int d = i * 32 + lane;
+                        x[e][i] = d < a.dv ? ldc<TC>(vr + d) : 0.f;
+                    }
                 }
             }
 #pragma unroll
@@ -319,7 +335,7 @@ __global__ void __launch_bounds__(AW * 32) kf_attn_window_kernel(WinArgs a) {
     }
 #pragma unroll
     for (int i = 0; i < VPL; i++) {
-        const int d = i * 32 + lane;
+        const int d = d_of(i);
         if (d < a.dv) sacc[warp * a.dv + d] = acc[i];
     }
     if (lane == 0) sml[warp * 2] = mx, sml[warp * 2 + 1] = l;
@@ -374,7 +390,7 @@ __global__ void kf_attn_window_merge_kernel(WinArgs a) {
 __device__ __forceinline__ float sig_f(float z) { return 1.f / (1.f + expf(-z)); }
 template <typename TC, int VPL>
 __global__ void __launch_bounds__(AW * 32) kf_attn_sigmoid_kernel(WinArgs a) {
-    extern __shared__ float sm[];
+    extern __shared__ __align__(16) float sm[];
     float* sq   = sm;         // [dk]
     float* sacc = sq + a.dk;  // [AW][dv]
     const int m = blockIdx.x, h = blockIdx.y, kh = h / (a.H / a.G);
@@ -552,7 +568,7 @@ extern "C" int kf_attn_window_ex(kf_ctx* ctx, void* out, int out_f32, int ldo, c
     if (window > 0) max_keys_hint = std::min(max_keys_hint, window) + (pool > 0 ? std::max(0, max_keys_hint - window) / pool : 0);
     int nsplit = 1;  // few (token, head) pairs and many keys (decoding): the keys are dealt to several CTAs so that the SMs are busy
     if (M * H < 2 * ctx->sm_count && max_keys_hint >= 4 * AW * 32)
-        nsplit = std::max(1, std::min(std::min(64, (2 * ctx->sm_count) / (M * H)), max_keys_hint / (2 * AW * 32)));
+        nsplit = std::max(1, std::min(std::min(64, (2 * ctx->sm_count) / (M * H)), max_keys_hint / (AW * 32)));
     if (nsplit > 1) {
         KF_REQUIRE(ctx, kf_ensure_attn_ws(ctx, (size_t)M * H * nsplit * (dv + 2) * sizeof(float)) == KF_OK, "attention workspace");
         a.ws = ctx->attn_ws;

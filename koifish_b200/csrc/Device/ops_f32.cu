@@ -143,48 +143,122 @@ struct PostArgs {
     const int32_t *pos, *slot;
     int cache;  // 1: dynamic shared memory holds the row of v, so its parts are read once
 };
-template <int SRC, typename TO>
+// V = 4: a thread takes four neighbouring entries per access (the row length and every row's address allow it), V = 1: one.
+template <int V>
+__device__ __forceinline__ void ldf(float (&v)[V], const float* p) {
+    if (V == 4) {
+        const float4 t = *reinterpret_cast<const float4*>(p);
+        v[0] = t.x, v[1 % V] = t.y, v[2 % V] = t.z, v[3 % V] = t.w;
+    } else {
+        v[0] = *p;
+    }
+}
+template <int V>
+__device__ __forceinline__ void stf(float* p, const float (&v)[V]) {
+    if (V == 4) *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1 % V], v[2 % V], v[3 % V]);
+    else *p = v[0];
+}
+template <int V>
+__device__ __forceinline__ void ldb(float (&v)[V], const uint16_t* p) {
+    if (V == 4) {
+        const uint2 t = *reinterpret_cast<const uint2*>(p);
+        v[0] = bf16lo(t.x), v[1 % V] = bf16hi(t.x), v[2 % V] = bf16lo(t.y), v[3 % V] = bf16hi(t.y);
+    } else {
+        v[0] = bf16_bits_to_f32(*p);
+    }
+}
+constexpr int kPostTop = 64;  // experts of a token whose places and weights are staged in shared memory
+template <int SRC, typename TO, int V>
 __global__ void kf_postnorm_kernel(PostArgs p) {
-    extern __shared__ float sv[];
+    extern __shared__ __align__(16) float sv[];
     __shared__ float red[32];
+    __shared__ int s_slot[kPostTop];
+    __shared__ float s_wgt[kPostTop];
     const int r = blockIdx.x;
-    auto val = [&](int i) -> float {
+    if (SRC == 1) {  // read once, so that the rows below are fetched side by side
+        for (int j = threadIdx.x; j < min(p.top, kPostTop); j += blockDim.x)
+            s_slot[j] = p.entry_slot[(size_t)r * p.top + j], s_wgt[j] = p.wgt[(size_t)r * p.top + j];
+        __syncthreads();
+    }
+    auto val = [&](float (&v)[V], int i) {
         if (SRC == 0) {
-            const float x = p.sa * p.a[(size_t)r * p.lda + i];
-            return p.b ? fmaf(p.sb, p.b[(size_t)r * p.ldb + i], x) : x;
+            ldf<V>(v, p.a + (size_t)r * p.lda + i);
+#pragma unroll
+            for (int k = 0; k < V; k++) v[k] *= p.sa;
+            if (p.b) {
+                float t[V];
+                ldf<V>(t, p.b + (size_t)r * p.ldb + i);
+#pragma unroll
+                for (int k = 0; k < V; k++) v[k] = fmaf(p.sb, t[k], v[k]);
+            }
+        } else if (SRC == 1) {
+            float sh[V];
+            if (p.shared) ldf<V>(sh, p.shared + (size_t)r * p.dim + i);
+#pragma unroll
+            for (int k = 0; k < V; k++) v[k] = 0.f;
+            const int n = min(p.top, kPostTop);
+#pragma unroll 4
+            for (int j = 0; j < n; j++) {
+                float t[V];
+                ldf<V>(t, p.y + (size_t)s_slot[j] * p.dim + i);
+#pragma unroll
+                for (int k = 0; k < V; k++) v[k] = fmaf(s_wgt[j], t[k], v[k]);
+            }
+            for (int j = kPostTop; j < p.top; j++) {
+                float t[V];
+                ldf<V>(t, p.y + (size_t)p.entry_slot[(size_t)r * p.top + j] * p.dim + i);
+#pragma unroll
+                for (int k = 0; k < V; k++) v[k] = fmaf(p.wgt[(size_t)r * p.top + j], t[k], v[k]);
+            }
+            if (p.shared)
+#pragma unroll
+                for (int k = 0; k < V; k++) v[k] += sh[k];
+        } else {
+            ldb<V>(v, p.table + (size_t)p.tokens[r] * p.dim + i);
         }
-        if (SRC == 1) {
-            float s = 0.f;
-            for (int j = 0; j < p.top; j++) s = fmaf(p.wgt[(size_t)r * p.top + j], p.y[(size_t)p.entry_slot[(size_t)r * p.top + j] * p.dim + i], s);
-            return p.shared ? s + p.shared[(size_t)r * p.dim + i] : s;
-        }
-        return bf16_bits_to_f32(p.table[(size_t)p.tokens[r] * p.dim + i]);
     };
     float ss = 0.f;
-    for (int i = threadIdx.x; i < p.dim; i += blockDim.x) {
-        const float v = val(i);
-        if (p.cache) sv[i] = v;  // read back by the same thread
-        ss = fmaf(v, v, ss);
+    for (int i = threadIdx.x * V; i < p.dim; i += blockDim.x * V) {
+        float v[V];
+        val(v, i);
+        if (p.cache) stf<V>(sv + i, v);  // read back by the same thread
+#pragma unroll
+        for (int k = 0; k < V; k++) ss = fmaf(v[k], v[k], ss);
     }
     ss = block_sum(ss, red);
     const float s = 1.0f / sqrtf(ss / (float)p.dim + p.eps);
     const float w1 = p.w_one ? p.w_add + bf16_bits_to_f32(p.w[0]) : 0.f;
     float* tail = p.shift ? p.tail + (size_t)p.slot[r] * p.tail_stride : nullptr;
     const bool first = p.shift && p.pos[r] == 0;
-    for (int i = threadIdx.x; i < p.dim; i += blockDim.x) {
+    for (int i = threadIdx.x * V; i < p.dim; i += blockDim.x * V) {
         float* q = p.res + (size_t)r * p.dim + i;
-        const float n = (p.cache ? sv[i] : val(i)) * s * (p.w_one ? w1 : p.w_add + bf16_bits_to_f32(p.w[i]));
-        const float x = SRC == 2 ? n : *q + p.mult * n;
-        *q = x;
-        float o = x;
-        if (p.shift) {
-            const float prev = first ? 0.f : tail[i];
-            o = fmaf(prev - x, bf16_bits_to_f32(p.shift[i]), x);
-            tail[i] = x;
+        float v[V], w[V], x[V];
+        if (p.cache) ldf<V>(v, sv + i);
+        else val(v, i);
+        if (!p.w_one) ldb<V>(w, p.w + i);
+        if (SRC != 2) ldf<V>(x, q);
+#pragma unroll
+        for (int k = 0; k < V; k++) {
+            const float n = v[k] * s * (p.w_one ? w1 : p.w_add + w[k]);
+            x[k] = SRC == 2 ? n : x[k] + p.mult * n;
         }
-        if (p.act) {
-            if (sizeof(TO) == 2) ((uint16_t*)p.act)[(size_t)r * p.dim + i] = f32_to_bf16_bits(o);
-            else ((float*)p.act)[(size_t)r * p.dim + i] = o;
+        stf<V>(q, x);
+        if (p.shift) {
+            float prev[V], sh[V];
+            ldb<V>(sh, p.shift + i);
+            ldf<V>(prev, tail + i);
+            stf<V>(tail + i, x);
+#pragma unroll
+            for (int k = 0; k < V; k++) x[k] = fmaf((first ? 0.f : prev[k]) - x[k], sh[k], x[k]);
+        }
+        if (!p.act) continue;
+        if (sizeof(TO) == 4) {
+            stf<V>((float*)p.act + (size_t)r * p.dim + i, x);
+        } else if (V == 4) {
+            const uint2 o = make_uint2(pack_bf16x2(x[0], x[1 % V]), pack_bf16x2(x[2 % V], x[3 % V]));
+            *reinterpret_cast<uint2*>((uint16_t*)p.act + (size_t)r * p.dim + i) = o;
+        } else {
+            ((uint16_t*)p.act)[(size_t)r * p.dim + i] = f32_to_bf16_bits(x[0]);
         }
     }
 }
@@ -192,9 +266,14 @@ template <int SRC>
 int launch_postnorm(kf_ctx* ctx, PostArgs& p, int act_f32, int rows) {
     const size_t smem = (size_t)p.dim * sizeof(float);
     p.cache = smem <= 32 * 1024 ? 1 : 0;
-    const int threads = rows <= 16 && p.dim >= 2048 ? 512 : 256;  // few rows: the row's loads go out side by side
-    if (act_f32) kf_postnorm_kernel<SRC, float><<<rows, threads, p.cache ? smem : 0, ctx->stream>>>(p);
-    else kf_postnorm_kernel<SRC, uint16_t><<<rows, threads, p.cache ? smem : 0, ctx->stream>>>(p);
+    const uintptr_t at = (uintptr_t)p.res | (uintptr_t)p.act | (uintptr_t)p.a | (uintptr_t)p.b | (uintptr_t)p.y | (uintptr_t)p.shared | (uintptr_t)p.tail;
+    const uintptr_t at2 = (uintptr_t)p.table | (p.w_one ? 0 : (uintptr_t)p.w) | (uintptr_t)p.shift;
+    const bool v4 = p.dim % 4 == 0 && p.lda % 4 == 0 && p.ldb % 4 == 0 && p.tail_stride % 4 == 0 && at % 16 == 0 && at2 % 8 == 0;
+    const int threads = v4 ? std::min(rows <= 16 ? 512 : 256, std::max(64, (p.dim / 4 + 31) / 32 * 32)) : 256;
+#define KF_PN(T, V) kf_postnorm_kernel<SRC, T, V><<<rows, threads, p.cache ? smem : 0, ctx->stream>>>(p)
+    if (act_f32) v4 ? KF_PN(float, 4) : KF_PN(float, 1);
+    else v4 ? KF_PN(uint16_t, 4) : KF_PN(uint16_t, 1);
+#undef KF_PN
     KF_LAUNCH_CHECK(ctx);
     return KF_OK;
 }
