@@ -568,7 +568,7 @@ extern "C" int kf_attn_window_ex(kf_ctx* ctx, void* out, int out_f32, int ldo, c
     if (window > 0) max_keys_hint = std::min(max_keys_hint, window) + (pool > 0 ? std::max(0, max_keys_hint - window) / pool : 0);
     int nsplit = 1;  // few (token, head) pairs and many keys (decoding): the keys are dealt to several CTAs so that the SMs are busy
     if (M * H < 2 * ctx->sm_count && max_keys_hint >= 4 * AW * 32)
-        nsplit = std::max(1, std::min(std::min(64, (2 * ctx->sm_count) / (M * H)), max_keys_hint / (AW * 32)));
+        nsplit = std::max(1, std::min(std::min(64, (2 * ctx->sm_count) / (M * H)), (max_keys_hint + AW * 32 - 1) / (AW * 32)));  // one 32-key step per warp
     if (nsplit > 1) {
         KF_REQUIRE(ctx, kf_ensure_attn_ws(ctx, (size_t)M * H * nsplit * (dv + 2) * sizeof(float)) == KF_OK, "attention workspace");
         a.ws = ctx->attn_ws;
