@@ -1,4 +1,4 @@
-"""Small random Gadilix models for the tests: layer cards, a config.json, weights drawn on the bf16 grid (optionally shaped so that a fault
+"""Small random Gadilix models for the tests: layer entries, a config.json, weights drawn on the bf16 grid (optionally shaped so that a fault
 shows), bf16 bit patterns, random token lists."""
 import numpy as np
 import torch
