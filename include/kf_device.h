@@ -462,6 +462,57 @@ int kf_attn_window_ex(kf_ctx* ctx, void* out_dev, int out_f32, int ldo, const fl
 int kf_attn_pooled_prefill(kf_ctx* ctx, void* out_bf16_dev, int ldo, const void* q_bf16_dev, const void* cache_dev, size_t slot_stride, int ring,
                            const void* sink_bf16_dev, const int32_t* pos_dev, const int32_t* slot_dev, int M, int n_head, int n_kv, int hd, float scale,
                            float softcap, int window, int pool, const float* head_gate_dev, int ldg, float out_scale);
+/* ---- stacks whose norm is n(x) = tanh(alpha x) w + b, entry by entry ----
+ * One step of the residual stream: x = res + scale * (what the call adds), out = n(x) in the activation type. */
+typedef struct kf_dyt_step {
+    float* res;                  /* [rows][dim], updated in place (left alone when row_idx is given) */
+    int rows, dim;
+    const void* scale_bf16;      /* [dim] factor on what is added, or NULL */
+    const void *w_bf16, *b_bf16; /* [dim]; w NULL: only the sum */
+    const void* alpha_bf16;      /* one number */
+    void* out;                   /* [rows][dim], or n_mix such planes `plane` elements apart */
+    int out_f32;
+    const int32_t* row_idx;      /* rows to take (device), or NULL */
+    /* token mixes (mu [n_mix][dim], or NULL): out plane s = h + (h' - h) mu_s, h = n(x), h' = n(x) of the sequence's previous token, zeros at position 0;
+     * the tail [slot][tail_stride] carries h from step to step */
+    int n_mix;
+    const void* mu_bf16;
+    size_t plane;
+    float* tail;
+    size_t tail_stride;
+    const int32_t *pos, *slot;
+} kf_dyt_step;
+/* adds float rows a [rows][lda] (NULL: nothing); with mu, every row is one token of a sequence of its own */
+int kf_dyt_residual(kf_ctx* ctx, const kf_dyt_step* s, const float* a_dev, int lda);
+/* adds sum_j wgt[m][j] * y_slots[entry_slot[m][j]], a slot of -1 standing for row m of pass (activation type; may be the buffer of out) */
+int kf_dyt_experts(kf_ctx* ctx, const kf_dyt_step* s, const float* y_slots_dev, const int32_t* entry_slot_dev, const float* wgt_dev, const void* pass_dev, int top);
+/* starts the stream: res[m] = table[token[m]] */
+int kf_dyt_embed(kf_ctx* ctx, const kf_dyt_step* s, const kf_tensor_desc* table, const int32_t* tokens_dev);
+/* the token mixes of n(res) for nseq sequences of T consecutive tokens each; res is only read */
+int kf_dyt_token_mix(kf_ctx* ctx, const kf_dyt_step* s, int nseq, int T);
+/* kf_moe_route's tables from softmax scores over experts + pass outputs: the choice runs over s + choice_bias inside the `keep` best of `groups` equal
+ * groups of adjacent outputs (a group ranks by its largest choice value), weights = s over (the chosen ones' sum + 1e-20); an entry that goes to
+ * one of the last `pass` outputs gets entry_slot -1, an unused slot gets slot_group -1 */
+int kf_moe_route_softmax_grouped(kf_ctx* ctx, int32_t* idx_dev, float* wgt_dev, int32_t* offsets_dev, int32_t* entry_slot_dev, int32_t* slot_row_dev,
+                                 int32_t* slot_group_dev, int32_t* work_dev, const float* logits_dev, int ldl, const void* choice_bias_bf16_dev, int M,
+                                 int experts, int pass, int top, int groups, int keep);
+/* kf_linear_grouped's two-weight form with y = g sigmoid(alpha g) (u + shift), g = min(W x, limit), u = clamp(W2 x, -limit, limit) (limit <= 0: no clamp) */
+int kf_linear_grouped_glu(kf_ctx* ctx, void* y_dev, int ldy, const void* const* w_table_dev, const void* const* w2_table_dev, int n_groups, int N, int K,
+                          const void* x_dev, int act_f32, int ldx, const int32_t* offsets_dev, const int32_t* slot_group_dev, const int32_t* src_row_dev,
+                          int slots, float limit, float alpha, float shift);
+/* y[i][m] = act_i(W_i x[i][m]) for n <= 8 bf16 weights of equal column count with inputs [M][ldx] and float outputs [M][rows of W_i] of their own (host arrays
+ * of device pointers); act: 0 none, 3 tanh (NULL: none) */
+int kf_linear_batch(kf_ctx* ctx, int n, float* const* y, const kf_tensor_desc* w, const void* const* x, const int* act, int act_f32, int ldx, int M);
+/* matrix-state recurrence whose read-out comes ahead of the write: o = S^T r + (r . (u * k)) v, S <- diag(exp(-exp(z + b))) S + k v^T */
+int kf_wkv_scan(kf_ctx* ctx, float* y_dev, int ldy, const float* r_dev, int ldr, const float* k_dev, int ldk, const float* v_dev, int ldv, const float* z_dev,
+                int ldz, const void* zbias_bf16_dev, const void* bonus_bf16_dev, float* state_dev, size_t state_stride, const int32_t* pos_dev,
+                const int32_t* slot_dev, int nseq, int T, int H, int dk, int dv);
+/* kf_qk_heads_prepare with norms that have no weight (unit_qk 1) and values blended with those of an earlier layer (v_first float [M][ld_first];
+ * v_blend NULL: this layer's values are copied there, else v = (1 - l) v + l v_first before caching) */
+int kf_qk_heads_prepare_ex(kf_ctx* ctx, float* x_dev, int ldx, int H, int G, int dk, int dv, const void* q_norm_bf16_dev, const void* k_norm_bf16_dev, int unit_qk,
+                           float eps, int rot_dims, const double* inv_freq_dev, float amp, int layout, float* v_first_dev, int ld_first,
+                           const void* v_blend_bf16_dev, void* cache_dev, int cache_f32, size_t slot_stride, int ring, int pool, int one_per_slot,
+                           void* q_bf16_out_dev, const int32_t* pos_dev, const int32_t* slot_dev, int M);
 
 #ifdef __cplusplus
 }

@@ -35,6 +35,12 @@ class ModelInfo(C.Structure):
                [(n, C.c_uint64) for n in ("weight_bytes", "kv_bytes", "block_weight_bytes_per_layer", "head_weight_bytes")]
 
 
+class DytStep(C.Structure):
+    _fields_ = [("res", C.c_void_p), ("rows", C.c_int), ("dim", C.c_int), ("scale_bf16", C.c_void_p), ("w_bf16", C.c_void_p), ("b_bf16", C.c_void_p),
+                ("alpha_bf16", C.c_void_p), ("out", C.c_void_p), ("out_f32", C.c_int), ("row_idx", C.c_void_p), ("n_mix", C.c_int), ("mu_bf16", C.c_void_p),
+                ("plane", C.c_size_t), ("tail", C.c_void_p), ("tail_stride", C.c_size_t), ("pos", C.c_void_p), ("slot", C.c_void_p)]
+
+
 # every symbol include/*.h declares, with its signature: (restype, [argtypes])
 _P, _I, _SZ, _U64, _F = C.c_void_p, C.c_int, C.c_size_t, C.c_uint64, C.c_float
 _DESCP = C.POINTER(TensorDesc)
@@ -151,6 +157,15 @@ SIGNATURES = {
     "kf_qk_heads_prepare": (_I, [_P, _P, _I, _I, _I, _I, _I, _P, _P, _F, _I, _P, _F, _I, _P, _I, _SZ, _I, _I, _I, _P, _P, _P, _I]),
     "kf_attn_window_ex": (_I, [_P, _P, _I, _I, _P, _I, _P, _I, _SZ, _I, _P, _P, _P, _I, _I, _I, _I, _I, _F, _F, _I, _I, _F, _I, _P, _I]),
     "kf_attn_pooled_prefill": (_I, [_P, _P, _I, _P, _P, _SZ, _I, _P, _P, _P, _I, _I, _I, _I, _F, _F, _I, _I, _P, _I, _F]),
+    "kf_dyt_residual": (_I, [_P, C.POINTER(DytStep), _P, _I]),
+    "kf_dyt_experts": (_I, [_P, C.POINTER(DytStep), _P, _P, _P, _P, _I]),
+    "kf_dyt_embed": (_I, [_P, C.POINTER(DytStep), _DESCP, _P]),
+    "kf_dyt_token_mix": (_I, [_P, C.POINTER(DytStep), _I, _I]),
+    "kf_moe_route_softmax_grouped": (_I, [_P, _P, _P, _P, _P, _P, _P, _P, _P, _I, _P, _I, _I, _I, _I, _I, _I]),
+    "kf_linear_grouped_glu": (_I, [_P, _P, _I, _P, _P, _I, _I, _I, _P, _I, _I, _P, _P, _P, _I, _F, _F, _F]),
+    "kf_linear_batch": (_I, [_P, _I, C.POINTER(_P), _DESCP, C.POINTER(_P), C.POINTER(_I), _I, _I, _I]),
+    "kf_wkv_scan": (_I, [_P, _P, _I, _P, _I, _P, _I, _P, _I, _P, _I, _P, _P, _P, _SZ, _P, _P, _I, _I, _I, _I, _I]),
+    "kf_qk_heads_prepare_ex": (_I, [_P, _P, _I, _I, _I, _I, _I, _P, _P, _I, _F, _I, _P, _F, _I, _P, _I, _P, _P, _I, _SZ, _I, _I, _I, _P, _P, _P, _I]),
     "kf_nccl_unique_id": (_I, [_P]),
     "kf_ctx_init_nccl": (_I, [_P, _P, _I, _I]),
     "kf_allreduce_bf16": (_I, [_P, _P, _SZ]),

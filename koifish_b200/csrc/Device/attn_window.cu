@@ -122,6 +122,10 @@ struct HeadsArgs {
     uint16_t* qb;  // given: q goes there as bf16 [M][H * dk] and x keeps the projection; NULL: q replaces it in x
     int ldx, H, G, dk, dv;
     const uint16_t *qw, *kw;  // bf16 [dk] or NULL (not normed)
+    int unit;                 // 1: without a weight every head of q and k is still divided by its root mean square
+    float* vfirst;            // [M][ldvf] float rows of G * dv, or NULL
+    int ldvf;
+    const uint16_t* vblend;   // vfirst given: NULL: v is copied there; a bf16 number l: v becomes (1 - l) v + l vfirst
     float eps, amp;
     int rot_dims, layout;
     const double* inv_freq;
@@ -159,11 +163,22 @@ __global__ void __launch_bounds__(HW * 32) kf_qk_heads_kernel(HeadsArgs a) {
         sx[d] = v, ss = fmaf(v, v, ss);
     }
     float f = 1.f;
-    if (w) f = 1.0f / sqrtf(warp_sum(ss) / (float)n + a.eps);
+    const bool unit = !w && a.unit && kind != 2;
+    if (w || unit) f = 1.0f / sqrtf(warp_sum(ss) / (float)n + a.eps);
     const int half = a.rot_dims >> 1;
     const bool rot = kind != 2 && half > 0;
     if (w)
         for (int d = lane; d < n; d += 32) sx[d] *= f * bf16_bits_to_f32(w[d]);
+    if (unit)
+        for (int d = lane; d < n; d += 32) sx[d] *= f;
+    if (kind == 2 && a.vfirst) {
+        float* vf = a.vfirst + (size_t)m * a.ldvf + hh * a.dv;
+        const float l = a.vblend ? bf16_bits_to_f32(*a.vblend) : 0.f;
+        for (int d = lane; d < n; d += 32) {
+            if (a.vblend) sx[d] = (1.f - l) * sx[d] + l * vf[d];
+            else vf[d] = sx[d];
+        }
+    }
     __syncwarp();
     TC* slot_rows = (TC*)a.cache + (size_t)a.slot[m] * a.slot_stride;
     const int coff = kind == 2 ? nk + hh * a.dv : hh * a.dk;  // this head's entries inside a cache row
@@ -514,16 +529,28 @@ extern "C" int kf_qk_prepare_ex(kf_ctx* ctx, float* x, int ldx, int nq, int nk, 
 extern "C" int kf_qk_heads_prepare(kf_ctx* ctx, float* x, int ldx, int H, int G, int dk, int dv, const void* q_norm_bf16, const void* k_norm_bf16, float eps, int rot_dims,
                                    const double* inv_freq_dev, float amp, int layout, void* cache, int cache_f32, size_t slot_stride, int ring, int pool,
                                    int one_per_slot, void* q_bf16_out, const int32_t* pos_dev, const int32_t* slot_dev, int M) {
+    return kf_qk_heads_prepare_ex(ctx, x, ldx, H, G, dk, dv, q_norm_bf16, k_norm_bf16, 0, eps, rot_dims, inv_freq_dev, amp, layout, nullptr, 0, nullptr, cache, cache_f32,
+                                  slot_stride, ring, pool, one_per_slot, q_bf16_out, pos_dev, slot_dev, M);
+}
+// The same with norms that have no weight (unit_qk 1: a head without a norm weight is still divided by its root mean square) and values that
+// are blended with those of an earlier layer: v_first float [M][ld_first >= G * dv]; v_blend NULL: this layer's values are copied there,
+// otherwise (a bf16 number l) its values become (1 - l) v + l v_first before they are cached.
+extern "C" int kf_qk_heads_prepare_ex(kf_ctx* ctx, float* x, int ldx, int H, int G, int dk, int dv, const void* q_norm_bf16, const void* k_norm_bf16, int unit_qk,
+                                      float eps, int rot_dims, const double* inv_freq_dev, float amp, int layout, float* v_first, int ld_first,
+                                      const void* v_blend_bf16, void* cache, int cache_f32, size_t slot_stride, int ring, int pool, int one_per_slot,
+                                      void* q_bf16_out, const int32_t* pos_dev, const int32_t* slot_dev, int M) {
     if (!ctx || !x || !cache || !pos_dev || !slot_dev) return KF_ERR_BAD_ARG;
     KF_REQUIRE(ctx, M >= 1 && H >= 1 && G >= 1 && dk >= 1 && dv >= 1 && dk <= 2048 && dv <= 2048 && ring >= 1 && ldx >= H * dk + G * (dk + dv), "shape");
     KF_REQUIRE(ctx, rot_dims >= 0 && rot_dims <= dk && rot_dims % 2 == 0 && (rot_dims == 0 || inv_freq_dev) && (layout == 0 || layout == 1), "rotation");
     KF_REQUIRE(ctx, pool >= 0 && (pool == 0 || ring >= pool), "the ring covers a pooled block");
+    KF_REQUIRE(ctx, v_first ? ld_first >= G * dv : !v_blend_bf16, "values to blend with");
     const int W = G * (dk + dv);
     KF_REQUIRE(ctx, slot_stride >= (size_t)ring * W, "slot stride");
     HeadsArgs a = {};
     a.x = x, a.qb = (uint16_t*)q_bf16_out, a.ldx = ldx, a.H = H, a.G = G, a.dk = dk, a.dv = dv, a.qw = (const uint16_t*)q_norm_bf16, a.kw = (const uint16_t*)k_norm_bf16;
     a.eps = eps, a.amp = amp, a.rot_dims = rot_dims, a.layout = layout, a.inv_freq = inv_freq_dev, a.cache = cache, a.slot_stride = slot_stride, a.ring = ring;
     a.pool = pool, a.pool_now = one_per_slot ? 1 : 0, a.pos = pos_dev, a.slot = slot_dev;
+    a.unit = unit_qk ? 1 : 0, a.vfirst = v_first, a.ldvf = ld_first, a.vblend = (const uint16_t*)v_blend_bf16;
     const dim3 grid(M, (H + 2 * G + HW - 1) / HW);
     const size_t smem = (size_t)HW * std::max(dk, dv) * sizeof(float);
     if (cache_f32) kf_qk_heads_kernel<float><<<grid, HW * 32, smem, ctx->stream>>>(a);

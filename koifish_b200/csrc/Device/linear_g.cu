@@ -4,7 +4,9 @@
 //     tensor-core matmul) or float (act_f32 = 1: a true 32-bit matmul, FMA by FMA, no reduced-precision mode);
 //   * "grouped" form for mixtures of experts: every output row (a slot) names the weight matrix it uses; slots of one expert are
 //     contiguous (offsets[e] .. offsets[e+1]) and may gather their input row through src_row;
-//   * DUAL form: two weight tables A, B of equal shape and y = silu(A x) * (B x), the gate / up pair of a gated feed-forward.
+//   * DUAL form: two weight tables A, B of equal shape and y = silu(A x) * (B x), the gate / up pair of a gated feed-forward, or its clamped
+//     form y = g sigmoid(alpha g) (u + shift) with g = min(A x, limit), u = clamp(B x, -limit, limit);
+//   * "batch" form for a handful of rows: several weights, each with an input and an output of its own, in one launch.
 // Two kernels: a warp-per-output GEMV for a handful of rows (decode: every weight row is read once, 16-byte loads when the row length
 // allows) and a 64 x 64 x 32 shared-memory tile kernel for panels (mma.sync m16n8k16 for bf16 activations, FFMA for float ones).
 // No reference equivalent: the reference's SLP::Forw hands every shape to cuBLASLt (src/Device/CUDA/NeuronFuse.cu:305-381).
@@ -26,11 +28,14 @@ struct LinArgs {
     const int32_t* slot_group;   // GEMV form: slot -> expert; nullptr: 0
     int M, N, K, ldx, ldy;
     int out_act;                 // DUAL or act != 0: 0 = float out, 1 = bf16 out, (float activations: float out)
-    int act;                     // single-weight form: 0 = none, 1 = gelu (tanh form), 2 = relu squared, applied to the result
+    int act;                     // single-weight form: 0 = none, 1 = gelu (tanh form), 2 = relu squared, 3 = tanh, applied to the result
+    int glu;                     // DUAL: 0 = silu(a) * b, 1 = the clamped form
+    float limit, alpha, shift;   // ... its constants (limit <= 0: not clamped)
 };
 __device__ __forceinline__ float lin_act(float v, int act) {
     if (act == 1) return 0.5f * v * (1.f + tanhf(0.7978845608028654f * (v + 0.044715f * v * v * v)));
     if (act == 2) return v > 0.f ? v * v : 0.f;
+    if (act == 3) return tanhf(v);
     return v;
 }
 
@@ -42,6 +47,11 @@ template <>
 __device__ __forceinline__ float ld_act<float>(const float* p) { return *p; }
 
 __device__ __forceinline__ float silu_f(float z) { return z / (1.f + expf(-z)); }
+__device__ __forceinline__ float lin_pair(const LinArgs& a, float g, float u) {
+    if (!a.glu) return silu_f(g) * u;
+    if (a.limit > 0.f) g = fminf(g, a.limit), u = fminf(fmaxf(u, -a.limit), a.limit);
+    return g / (1.f + expf(-a.alpha * g)) * (u + a.shift);
+}
 
 // ------------------------------------------------------------------------------------------------------------------ GEMV (few slots)
 // one warp per (slot, output n): lanes stride over k, fixed butterfly reduction -> deterministic.
@@ -52,6 +62,7 @@ __global__ void __launch_bounds__(256) kf_lin_gemv_kernel(LinArgs a) {
     const int slot = blockIdx.y;
     if (n >= a.N) return;
     const int g   = a.slot_group ? a.slot_group[slot] : 0;
+    if (g < 0) return;  // a slot that no token uses
     const int row = a.src_row ? a.src_row[slot] : slot;
     const uint16_t* w0 = (a.Wt0 ? a.Wt0[g] : a.W0) + (size_t)n * a.K;
     const uint16_t* w1 = DUAL ? (a.Wt1 ? a.Wt1[g] : a.W1) + (size_t)n * a.K : nullptr;
@@ -91,12 +102,59 @@ __global__ void __launch_bounds__(256) kf_lin_gemv_kernel(LinArgs a) {
     s0 = warp_sum(s0);
     if (DUAL) s1 = warp_sum(s1);
     if (lane == 0) {
-        const float r = DUAL ? silu_f(s0) * s1 : lin_act(s0, a.act);
+        const float r = DUAL ? lin_pair(a, s0, s1) : lin_act(s0, a.act);
         if ((DUAL || a.act) && a.out_act == 1)
             ((uint16_t*)a.y)[(size_t)slot * a.ldy + n] = f32_to_bf16_bits(r);
         else
             ((float*)a.y)[(size_t)slot * a.ldy + n] = r;
     }
+}
+
+// Several independent products of one reduction length, each with its own weight, input and output, for a handful of rows: a warp per
+// (row, output) as above; blockIdx.x walks the outputs of all of them one after the other.
+constexpr int kBatchMax = 8;
+struct BatchArgs {
+    const uint16_t* W[kBatchMax];
+    const void* x[kBatchMax];
+    float* y[kBatchMax];
+    int N[kBatchMax], ldy[kBatchMax], act[kBatchMax], first[kBatchMax + 1];  // first: the block at which a product starts
+    int n, K, ldx;
+};
+template <typename TA>
+__global__ void __launch_bounds__(256) kf_lin_gemv_batch_kernel(BatchArgs a) {
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, row = blockIdx.y;
+    int j = 0;
+#pragma unroll
+    for (int i = 1; i < kBatchMax; i++)
+        if (i < a.n && (int)blockIdx.x >= a.first[i]) j = i;
+    const int n = ((int)blockIdx.x - a.first[j]) * 8 + warp;
+    if (n >= a.N[j]) return;
+    const uint16_t* w = a.W[j] + (size_t)n * a.K;
+    const TA* x = (const TA*)a.x[j] + (size_t)row * a.ldx;
+    float s = 0.f;
+    if ((a.K % 8 == 0) && (a.ldx % 8 == 0) && (((uintptr_t)w & 15) == 0) && (((uintptr_t)x & 15) == 0)) {
+#pragma unroll 4
+        for (int k = lane * 8; k < a.K; k += 256) {
+            const uint4 wv = *reinterpret_cast<const uint4*>(w + k);
+            const uint32_t wq[4] = {wv.x, wv.y, wv.z, wv.w};
+            float xv[8];
+            if (sizeof(TA) == 2) {
+                const uint4 xq4 = *reinterpret_cast<const uint4*>((const uint16_t*)x + k);
+                const uint32_t xq[4] = {xq4.x, xq4.y, xq4.z, xq4.w};
+#pragma unroll
+                for (int i = 0; i < 4; i++) xv[2 * i] = bf16lo(xq[i]), xv[2 * i + 1] = bf16hi(xq[i]);
+            } else {
+                const float4 f0 = *reinterpret_cast<const float4*>((const float*)x + k), f1 = *reinterpret_cast<const float4*>((const float*)x + k + 4);
+                xv[0] = f0.x, xv[1] = f0.y, xv[2] = f0.z, xv[3] = f0.w, xv[4] = f1.x, xv[5] = f1.y, xv[6] = f1.z, xv[7] = f1.w;
+            }
+#pragma unroll
+            for (int i = 0; i < 4; i++) s = fmaf(bf16lo(wq[i]), xv[2 * i], s), s = fmaf(bf16hi(wq[i]), xv[2 * i + 1], s);
+        }
+    } else {
+        for (int k = lane; k < a.K; k += 32) s = fmaf(bf16_bits_to_f32(w[k]), ld_act<TA>(x + k), s);
+    }
+    s = warp_sum(s);
+    if (lane == 0) a.y[j][(size_t)row * a.ldy[j] + n] = lin_act(s, a.act[j]);
 }
 
 // ------------------------------------------------------------------------------------------------------------------ tile kernel
@@ -244,7 +302,7 @@ __global__ void __launch_bounds__(256) kf_lin_tile_kernel(LinArgs a) {
     auto store = [&](int r, int n, float v0, float v1) {
         const int s = m0 + r;
         if (s >= hi || n >= a.N) return;
-        const float v = DUAL ? silu_f(v0) * v1 : lin_act(v0, a.act);
+        const float v = DUAL ? lin_pair(a, v0, v1) : lin_act(v0, a.act);
         if ((DUAL || a.act) && a.out_act == 1)
             ((uint16_t*)a.y)[(size_t)s * a.ldy + n] = f32_to_bf16_bits(v);
         else
@@ -340,4 +398,52 @@ extern "C" int kf_linear_grouped_act(kf_ctx* ctx, void* y, int ldy, const void* 
     a.Wt0 = (const uint16_t* const*)w_table, a.x = x, a.y = y, a.M = slots, a.N = N, a.K = K;
     a.ldx = ldx, a.ldy = ldy, a.offsets = offsets, a.slot_group = slot_group, a.src_row = src_row, a.out_act = act_f32 ? 0 : 1, a.act = act;
     return dispatch(ctx, a, slots, n_groups, slots <= kGemvMaxSlots, false, act_f32);
+}
+// kf_linear_grouped's two-weight form with the clamped gate: y = g sigmoid(alpha g) (u + shift), g = min(W x, limit), u = clamp(W2 x, -limit,
+// limit) (limit <= 0: not clamped), written in the activation type.  A slot whose slot_group is -1 is left out.
+extern "C" int kf_linear_grouped_glu(kf_ctx* ctx, void* y, int ldy, const void* const* w_table, const void* const* w2_table, int n_groups, int N, int K,
+                                     const void* x, int act_f32, int ldx, const int32_t* offsets, const int32_t* slot_group, const int32_t* src_row, int slots,
+                                     float limit, float alpha, float shift) {
+    if (!ctx || !y || !w_table || !w2_table || !x || !offsets || !slot_group) return KF_ERR_BAD_ARG;
+    KF_REQUIRE(ctx, n_groups >= 1 && N >= 1 && K >= 1 && slots >= 1 && ldx >= K && ldy >= N, "shape");
+    LinArgs a = {};
+    a.Wt0 = (const uint16_t* const*)w_table, a.Wt1 = (const uint16_t* const*)w2_table, a.x = x, a.y = y, a.M = slots, a.N = N, a.K = K;
+    a.ldx = ldx, a.ldy = ldy, a.offsets = offsets, a.slot_group = slot_group, a.src_row = src_row, a.out_act = act_f32 ? 0 : 1;
+    a.glu = 1, a.limit = limit, a.alpha = alpha, a.shift = shift;
+    return dispatch(ctx, a, slots, n_groups, slots <= kGemvMaxSlots, true, act_f32);
+}
+// y[i][m] = act_i(W_i x[i][m]) for n <= 8 bf16 weights with the same number of columns, each with an input [M][ldx] and a float output [M][rows of
+// W_i] of its own; act: 0 none, 3 tanh (host array, NULL: none).  A handful of rows: one launch; panels: one matmul per weight.
+extern "C" int kf_linear_batch(kf_ctx* ctx, int n, float* const* y, const kf_tensor_desc* w, const void* const* x, const int* act, int act_f32, int ldx, int M) {
+    if (!ctx || !y || !w || !x) return KF_ERR_BAD_ARG;
+    KF_REQUIRE(ctx, n >= 1 && n <= kBatchMax && M >= 1, "1 .. 8 weights");
+    for (int i = 0; i < n; i++) {
+        KF_REQUIRE(ctx, y[i] && x[i] && w[i].type == KF_T_BF16 && w[i].rows >= 1 && w[i].cols == w[0].cols && ldx >= w[i].cols, "bf16 weights, equal columns");
+        KF_REQUIRE(ctx, !act || act[i] == 0 || act[i] == 3, "act");
+    }
+    if (M > kGemvMaxSlots) {
+        for (int i = 0; i < n; i++) {
+            int rc;
+            if (act && act[i]) {
+                LinArgs a = {};
+                a.W0 = (const uint16_t*)w[i].data_dev, a.x = x[i], a.y = y[i], a.M = M, a.N = w[i].rows, a.K = w[i].cols, a.ldx = ldx, a.ldy = w[i].rows, a.act = act[i];
+                rc = dispatch(ctx, a, M, 1, w[i].rows <= 64 && w[i].cols >= 512, false, act_f32);
+            } else {
+                rc = kf_linear_g(ctx, y[i], w[i].rows, &w[i], x[i], act_f32, ldx, M);
+            }
+            if (rc) return rc;
+        }
+        return KF_OK;
+    }
+    BatchArgs a = {};
+    a.n = n, a.K = w[0].cols, a.ldx = ldx;
+    for (int i = 0; i < n; i++) {
+        a.W[i] = (const uint16_t*)w[i].data_dev, a.x[i] = x[i], a.y[i] = y[i], a.N[i] = a.ldy[i] = w[i].rows, a.act[i] = act ? act[i] : 0;
+        a.first[i + 1] = a.first[i] + (w[i].rows + 7) / 8;
+    }
+    const dim3 grid(a.first[n], M);
+    if (act_f32) kf_lin_gemv_batch_kernel<float><<<grid, 256, 0, ctx->stream>>>(a);
+    else kf_lin_gemv_batch_kernel<uint16_t><<<grid, 256, 0, ctx->stream>>>(a);
+    KF_LAUNCH_CHECK(ctx);
+    return KF_OK;
 }

@@ -2,8 +2,10 @@
 //   (1) matrix-state recurrences with a decay per key channel: per head an fp32 state S [dk x dv] and, per token,
 //           S <- diag(g_t) S ;  then either   S <- S + k_t v_t^T                                   (gated linear attention)
 //                                     or      u = beta_t (v_t - S^T k_t),  S <- S + k_t u^T        (gated delta rule)
-//       and o_t = S^T q_t, taken after the write of token t.  The decay is formed in fp32 from a logit z while the
-//       token is staged: g = sigmoid(z + b)^(1/tau), or g = exp(-exp(A_h) softplus(z + b)).  q and k may be made unit vectors per head.
+//       and o_t = S^T q_t, taken after the write of token t; or the read-out comes FIRST and sees the token through a bonus,
+//           o_t = S^T q_t + (q_t . (u * k_t)) v_t,  then  S <- diag(g_t) S + k_t v_t^T               (time mixing with a bonus)
+//       The decay is formed in fp32 from a logit z while the token is staged: g = sigmoid(z + b)^(1/tau), g = exp(-exp(A_h) softplus(z + b)),
+//       or g = exp(-exp(z + b)).  q and k may be made unit vectors per head.
 //   (2) a real-gated linear recurrent unit over channels: block-diagonal gate matmuls r, i = sigmoid(W u_b + b), decay
 //       a = exp(-c r softplus(lam)), state s <- a s + sqrt(1 - a^2) i u, output s * y.
 // State lives in fp32 per (sequence slot, layer) and persists between calls; a slot whose first staged token has position 0 starts
@@ -33,8 +35,8 @@ struct ScanArgs {
     const int32_t *pos, *slot;
     int T, H, G, dk, dv;
     int R, PB, TB, dkp;      // dkp: padded length of a staged row
-    int delta;               // 1: delta-rule write, 0: plain outer-product write
-    int decay_kind;          // 0: sigmoid(z + b)^(1/tau) ; 1: exp(-exp(A_h) softplus(z + b))
+    int decay_kind;          // 0: sigmoid(z + b)^(1/tau) ; 1: exp(-exp(A_h) softplus(z + b)) ; 2: exp(-exp(z + b))
+    const uint16_t* bonus;   // bf16 [H * dk] (RULE 2)
     int unit_qk;             // q, k divided by sqrt(sum x^2 + unit_eps) per head
     int z_head;              // 1: one decay per head and token (z: [H], zbias: [H]) shared by the head's key channels
     float inv_tau, q_scale, unit_eps;
@@ -45,9 +47,11 @@ struct ScanArgs {
 // (normalised there), the decay (formed there), v, beta.  FULL (dk == R * NPT): a thread's slice of k, q and the decay is NPT / 4 16-byte
 // shared loads each and nothing is bounds-checked; otherwise rows beyond dk read k = q = 0 and leave their (zero) state alone.
 constexpr int NPT_MAX = 16;
-template <bool DELTA, bool FULL, int NPT>
+// RULE 0: plain outer-product write; 1: delta-rule write; 2: read-out ahead of the write, with a bonus.
+template <int RULE, bool FULL, int NPT>
 __global__ void __launch_bounds__(256) kf_gated_scan_kernel(ScanArgs a) {
     extern __shared__ __align__(16) float sm[];
+    constexpr bool DELTA = RULE == 1, BONUS = RULE == 2;
     // staged rows are padded by 4 floats after every 16: the R lanes of a column read slices 20 floats apart, which fall into different
     // banks (slices exactly 16 apart would collide two by two)
     const int dk = a.dk, TB = a.TB, PB = a.PB, R = a.R, dkp = a.dkp;
@@ -57,7 +61,7 @@ __global__ void __launch_bounds__(256) kf_gated_scan_kernel(ScanArgs a) {
     float* sG = sQ + TB * dkp;       // [TB][dkp]
     float* sV = sG + TB * dkp;       // [TB][PB]
     float* sB = sV + TB * PB;        // [TB]
-    float* sKQ = sB + TB;            // [TB] k . q of the staged (normalised, scaled) rows: the delta rule's read-out needs it
+    float* sKQ = sB + TB;            // [TB] k . q of the staged (normalised, scaled) rows: the delta rule's read-out needs it; RULE 2: (u * k) . q
     const int h = blockIdx.x, seq = blockIdx.y, p0 = blockIdx.z * PB;
     const int kh = h / (a.H / a.G);
     const int tid = threadIdx.x, pl = tid / R, r = tid - pl * R, p = p0 + pl;
@@ -69,6 +73,9 @@ __global__ void __launch_bounds__(256) kf_gated_scan_kernel(ScanArgs a) {
 #pragma unroll
     for (int i = 0; i < NPT; i++) S[i] = (live && n0 + i < dk && !fresh) ? st[n0 + i] : 0.f;
     const float Aexp = a.decay_kind == 1 ? expf(bf16_bits_to_f32(a.A_log[h])) : 0.f;
+    auto decay = [&](float z) {
+        return a.decay_kind == 2 ? expf(-expf(z)) : a.decay_kind == 1 ? expf(-Aexp * softplus_f(z)) : expf(log_sigmoid_f(z) * a.inv_tau);
+    };
     const bool zh = a.z_head != 0;  // one decay per head and token: formed once per staged token (sG[tt]), not per key channel
     const int warp = tid >> 5, lane = tid & 31, nwarp = blockDim.x >> 5;
     for (int t0 = 0; t0 < a.T; t0 += TB) {
@@ -93,14 +100,14 @@ __global__ void __launch_bounds__(256) kf_gated_scan_kernel(ScanArgs a) {
                 if (i < nt * dk) {
                     const int tt = i / dk, o = tt * dkp + ix(i - tt * dk);
                     sK[o] = kv[e], sQ[o] = qv[e];
-                    if (!zh) sG[o] = a.decay_kind == 1 ? expf(-Aexp * softplus_f(zv[e])) : expf(log_sigmoid_f(zv[e]) * a.inv_tau);
+                    if (!zh) sG[o] = decay(zv[e]);
                 }
             }
         }
         if (zh)
             for (int i = tid; i < nt; i += blockDim.x) {
                 const float z = a.z[(size_t)(m0 + t0 + i) * a.ldz + h] + (a.zbias ? bf16_bits_to_f32(a.zbias[h]) : 0.f);
-                sG[i] = a.decay_kind == 1 ? expf(-Aexp * softplus_f(z)) : expf(log_sigmoid_f(z) * a.inv_tau);
+                sG[i] = decay(z);
             }
         for (int i0 = tid; i0 < nt * PB; i0 += 4 * blockDim.x) {
             float vv[4];
@@ -130,9 +137,9 @@ __global__ void __launch_bounds__(256) kf_gated_scan_kernel(ScanArgs a) {
                 const float qn = sQ[tt * dkp + ix(n)] * fq, kn = sK[tt * dkp + ix(n)] * fk;
                 sQ[tt * dkp + ix(n)] = qn;
                 if (a.unit_qk) sK[tt * dkp + ix(n)] = kn;
-                kq = fmaf(kn, qn, kq);
+                kq = fmaf(BONUS ? bf16_bits_to_f32(a.bonus[h * dk + n]) * kn : kn, qn, kq);
             }
-            if (DELTA) {
+            if (DELTA || BONUS) {
                 kq = warp_sum(kq);
                 if (lane == 0) sKQ[tt] = kq;
             }
@@ -192,12 +199,13 @@ __global__ void __launch_bounds__(256) kf_gated_scan_kernel(ScanArgs a) {
             float c[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
             for (int i = 0; i < NPT; i++) {
-                S[i]     = fmaf(gg[i], S[i], kk[i] * w);
-                c[i & 3] = fmaf(S[i], qq[i], c[i & 3]);
+                if (BONUS) c[i & 3] = fmaf(S[i], qq[i], c[i & 3]);
+                S[i] = fmaf(gg[i], S[i], kk[i] * w);
+                if (!BONUS) c[i & 3] = fmaf(S[i], qq[i], c[i & 3]);
             }
             float acc = (c[0] + c[1]) + (c[2] + c[3]);
             for (int o = R >> 1; o > 0; o >>= 1) acc += __shfl_xor_sync(0xffffffffu, acc, o);
-            if (live && r == 0) a.y[(size_t)(m0 + t0 + tt) * a.ldy + h * a.dv + p] = acc;
+            if (live && r == 0) a.y[(size_t)(m0 + t0 + tt) * a.ldy + h * a.dv + p] = BONUS ? fmaf(sKQ[tt], w, acc) : acc;
         }
     }
     if (live) {
@@ -427,22 +435,8 @@ extern "C" int kf_mingru(kf_ctx* ctx, void* out, int out_f32, int ldo, const flo
     return KF_OK;
 }
 
-// Matrix-state recurrence over nseq x T tokens (see the head of this file).  q, k: float rows with G kv heads of dk entries at row strides
-// ldq / ldk; v: H heads of dv entries; z: decay logits H x dk (+ bf16 bias zbias or NULL); beta_logit: H per token (delta rule only).
-// decay_kind 0: g = sigmoid(z + b)^(1/tau); 1: g = exp(-exp(A_log[h]) softplus(z + b)).  state: float [slot][H][dv][dk].
-// decay_per_head 1: z holds ONE logit per head and token ([H] at row stride ldz, zbias [H]); every key channel of the head decays alike.
-extern "C" int kf_gated_scan_ex(kf_ctx* ctx, float* y, int ldy, const float* q, int ldq, const float* k, int ldk, const float* v, int ldv, const float* z,
-                             int ldz, const void* zbias_bf16, const void* A_log_bf16, const float* beta_logit, int ldb, float* state, size_t state_stride,
-                             const int32_t* pos_dev, const int32_t* slot_dev, int nseq, int T, int H, int G, int dk, int dv, int delta, int decay_kind,
-                             float tau, int unit_qk, float unit_eps, float q_scale, int decay_per_head) {
-    if (!ctx || !y || !q || !k || !v || !z || !state || !pos_dev || !slot_dev) return KF_ERR_BAD_ARG;
-    KF_REQUIRE(ctx, nseq >= 1 && T >= 1 && H >= 1 && G >= 1 && H % G == 0 && dk >= 1 && dv >= 1 && dk <= 32 * NPT_MAX, "key size <= 512, kv heads divide heads");
-    KF_REQUIRE(ctx, (!delta || beta_logit) && (decay_kind == 0 ? tau > 0.f : A_log_bf16 != nullptr) && state_stride >= (size_t)H * dk * dv, "arguments");
-    ScanArgs a = {};
-    a.y = y, a.ldy = ldy, a.q = q, a.k = k, a.v = v, a.z = z, a.beta = beta_logit, a.ldq = ldq, a.ldk = ldk, a.ldv = ldv, a.ldz = ldz, a.ldb = ldb;
-    a.zbias = (const uint16_t*)zbias_bf16, a.A_log = (const uint16_t*)A_log_bf16, a.state = state, a.state_stride = state_stride;
-    a.pos = pos_dev, a.slot = slot_dev, a.T = T, a.H = H, a.G = G, a.dk = dk, a.dv = dv, a.delta = delta, a.decay_kind = decay_kind;
-    a.unit_qk = unit_qk, a.inv_tau = decay_kind == 0 ? 1.f / tau : 0.f, a.q_scale = q_scale, a.unit_eps = unit_eps, a.z_head = decay_per_head ? 1 : 0;
+static int scan_launch(kf_ctx* ctx, ScanArgs& a, int nseq, int rule) {
+    const int T = a.T, H = a.H, dk = a.dk, dv = a.dv;
     // rows of a state column per lane: 16, or 8 for keys of up to 128 entries (a shorter dependent chain per token, twice the lanes per column)
     const int NPT = (dk <= 128 && dk % 8 == 0 && dk >= 16) ? 8 : 16;
     int R = 1;
@@ -461,17 +455,48 @@ extern "C" int kf_gated_scan_ex(kf_ctx* ctx, float* y, int ldy, const float* q, 
     const bool full = dk == R * NPT;
 #define KF_SCAN(D, F, N) kf_gated_scan_kernel<D, F, N><<<grid, threads, smem, ctx->stream>>>(a)
 #define KF_SCAN_N(D, F) (NPT == 8 ? KF_SCAN(D, F, 8) : KF_SCAN(D, F, 16))
-    if (delta) {
-        if (full) KF_SCAN_N(true, true);
-        else KF_SCAN_N(true, false);
-    } else {
-        if (full) KF_SCAN_N(false, true);
-        else KF_SCAN_N(false, false);
-    }
+#define KF_SCAN_R(D) (full ? KF_SCAN_N(D, true) : KF_SCAN_N(D, false))
+    if (rule == 1) KF_SCAN_R(1);
+    else if (rule == 2) KF_SCAN_R(2);
+    else KF_SCAN_R(0);
+#undef KF_SCAN_R
 #undef KF_SCAN_N
 #undef KF_SCAN
     KF_LAUNCH_CHECK(ctx);
     return KF_OK;
+}
+
+// Matrix-state recurrence over nseq x T tokens (see the head of this file).  q, k: float rows with G kv heads of dk entries at row strides
+// ldq / ldk; v: H heads of dv entries; z: decay logits H x dk (+ bf16 bias zbias or NULL); beta_logit: H per token (delta rule only).
+// decay_kind 0: g = sigmoid(z + b)^(1/tau); 1: g = exp(-exp(A_log[h]) softplus(z + b)).  state: float [slot][H][dv][dk].
+// decay_per_head 1: z holds ONE logit per head and token ([H] at row stride ldz, zbias [H]); every key channel of the head decays alike.
+extern "C" int kf_gated_scan_ex(kf_ctx* ctx, float* y, int ldy, const float* q, int ldq, const float* k, int ldk, const float* v, int ldv, const float* z,
+                             int ldz, const void* zbias_bf16, const void* A_log_bf16, const float* beta_logit, int ldb, float* state, size_t state_stride,
+                             const int32_t* pos_dev, const int32_t* slot_dev, int nseq, int T, int H, int G, int dk, int dv, int delta, int decay_kind,
+                             float tau, int unit_qk, float unit_eps, float q_scale, int decay_per_head) {
+    if (!ctx || !y || !q || !k || !v || !z || !state || !pos_dev || !slot_dev) return KF_ERR_BAD_ARG;
+    KF_REQUIRE(ctx, nseq >= 1 && T >= 1 && H >= 1 && G >= 1 && H % G == 0 && dk >= 1 && dv >= 1 && dk <= 32 * NPT_MAX, "key size <= 512, kv heads divide heads");
+    KF_REQUIRE(ctx, (!delta || beta_logit) && (decay_kind == 0 ? tau > 0.f : A_log_bf16 != nullptr) && state_stride >= (size_t)H * dk * dv, "arguments");
+    ScanArgs a = {};
+    a.y = y, a.ldy = ldy, a.q = q, a.k = k, a.v = v, a.z = z, a.beta = beta_logit, a.ldq = ldq, a.ldk = ldk, a.ldv = ldv, a.ldz = ldz, a.ldb = ldb;
+    a.zbias = (const uint16_t*)zbias_bf16, a.A_log = (const uint16_t*)A_log_bf16, a.state = state, a.state_stride = state_stride;
+    a.pos = pos_dev, a.slot = slot_dev, a.T = T, a.H = H, a.G = G, a.dk = dk, a.dv = dv, a.decay_kind = decay_kind;
+    a.unit_qk = unit_qk, a.inv_tau = decay_kind == 0 ? 1.f / tau : 0.f, a.q_scale = q_scale, a.unit_eps = unit_eps, a.z_head = decay_per_head ? 1 : 0;
+    return scan_launch(ctx, a, nseq, delta ? 1 : 0);
+}
+// Time mixing with a bonus over nseq x T tokens: per head o_t = S^T r_t + (r_t . (u * k_t)) v_t, then S <- diag(g_t) S + k_t v_t^T with the decay
+// g = exp(-exp(z + b)) per key channel.  r, k, z: float rows of H heads x dk; v, y: H heads x dv; zbias, bonus: bf16 [H * dk] (zbias may be
+// NULL); state: float [slot][H][dv][dk], started from zero at position 0.
+extern "C" int kf_wkv_scan(kf_ctx* ctx, float* y, int ldy, const float* r, int ldr, const float* k, int ldk, const float* v, int ldv, const float* z, int ldz,
+                           const void* zbias_bf16, const void* bonus_bf16, float* state, size_t state_stride, const int32_t* pos_dev, const int32_t* slot_dev,
+                           int nseq, int T, int H, int dk, int dv) {
+    if (!ctx || !y || !r || !k || !v || !z || !bonus_bf16 || !state || !pos_dev || !slot_dev) return KF_ERR_BAD_ARG;
+    KF_REQUIRE(ctx, nseq >= 1 && T >= 1 && H >= 1 && dk >= 1 && dv >= 1 && dk <= 32 * NPT_MAX && state_stride >= (size_t)H * dk * dv, "key size <= 512");
+    ScanArgs a = {};
+    a.y = y, a.ldy = ldy, a.q = r, a.k = k, a.v = v, a.z = z, a.ldq = ldr, a.ldk = ldk, a.ldv = ldv, a.ldz = ldz;
+    a.zbias = (const uint16_t*)zbias_bf16, a.bonus = (const uint16_t*)bonus_bf16, a.state = state, a.state_stride = state_stride;
+    a.pos = pos_dev, a.slot = slot_dev, a.T = T, a.H = a.G = H, a.dk = dk, a.dv = dv, a.decay_kind = 2, a.q_scale = 1.f;
+    return scan_launch(ctx, a, nseq, 2);
 }
 
 extern "C" int kf_gated_scan(kf_ctx* ctx, float* y, int ldy, const float* q, int ldq, const float* k, int ldk, const float* v, int ldv, const float* z,

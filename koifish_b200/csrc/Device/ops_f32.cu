@@ -333,6 +333,179 @@ __global__ void __launch_bounds__(256) kf_residual_prenorm_kernel(float* __restr
         else ((float*)act_out)[(size_t)r * dim + i] = v;
     }
 }
+// ---- steps of a stack whose norm is a saturating function of each entry, n(x) = tanh(alpha x) w + b: no statistics over the row, so every
+// step between two matmuls is entry by entry and any number of CTAs can share a row ------------------------------------------------------
+// Residual step:  x = res + scale * v (scale per entry, or none),  out = n(x) in the activation type;  v is
+//   SRC 0: a float row (NULL: nothing is added);  SRC 1: sum_j wgt[j] * y[entry_slot[j]], where an entry without a slot (-1) stands for the
+//   token's row of `pass`;  SRC 2: a row of a bf16 table, which starts the stream (res = the row).
+// row_idx: rows to take, res is then left alone.  mu (rows that are one token each of different sequences): instead of n(x), n_mix rows
+// h + (h' - h) mu_s one plane apart, h = n(x), h' = the row the sequence's previous token left in its tail (zeros at position 0); the tail
+// takes h.  `pass` may be `out`: a thread reads its own entries first.
+struct DytArgs {
+    float* res;
+    int dim;
+    const uint16_t *scale, *w, *b, *alpha;
+    void* out;
+    const int32_t* row_idx;
+    const uint16_t* mu;
+    int n_mix;
+    size_t plane;
+    float* tail;
+    size_t tail_stride;
+    const int32_t *pos, *slot;
+    const float* a;
+    int lda;
+    const float *y, *wgt;
+    const int32_t* entry_slot;
+    const void* pass;
+    int top;
+    const uint16_t* table;
+    const int32_t* tokens;
+    int T;  // token mix: tokens per sequence
+};
+template <typename TO, int V>
+__device__ __forceinline__ void st_act(TO* p, const float (&v)[V]) {
+    if (sizeof(TO) == 4) {
+        stf<V>((float*)p, v);
+    } else if (V == 4) {
+        *reinterpret_cast<uint2*>((uint16_t*)p) = make_uint2(pack_bf16x2(v[0], v[1 % V]), pack_bf16x2(v[2 % V], v[3 % V]));
+    } else {
+        *(uint16_t*)p = f32_to_bf16_bits(v[0]);
+    }
+}
+template <typename TO, int V>
+__device__ __forceinline__ void ld_actv(float (&v)[V], const TO* p) {
+    if (sizeof(TO) == 4) ldf<V>(v, (const float*)p);
+    else ldb<V>(v, (const uint16_t*)p);
+}
+template <int SRC, typename TO, int V>
+__global__ void __launch_bounds__(128) kf_dyt_step_kernel(DytArgs p) {
+    const int r = blockIdx.y, i = (blockIdx.x * blockDim.x + threadIdx.x) * V;
+    if (i >= p.dim) return;
+    const int src = p.row_idx ? p.row_idx[r] : r;
+    float v[V], x[V];
+#pragma unroll
+    for (int k = 0; k < V; k++) v[k] = 0.f;
+    if (SRC != 2) ldf<V>(x, p.res + (size_t)src * p.dim + i);
+    if (SRC == 0) {
+        if (p.a) ldf<V>(v, p.a + (size_t)src * p.lda + i);
+    } else if (SRC == 1) {
+        const int32_t* es = p.entry_slot + (size_t)src * p.top;
+        const float* wg   = p.wgt + (size_t)src * p.top;
+#pragma unroll 4
+        for (int j = 0; j < p.top; j++) {
+            const int sl = es[j];
+            const float wj = wg[j];
+            float t[V];
+            if (sl >= 0) ldf<V>(t, p.y + (size_t)sl * p.dim + i);
+            else ld_actv<TO, V>(t, (const TO*)p.pass + (size_t)src * p.dim + i);
+#pragma unroll
+            for (int k = 0; k < V; k++) v[k] = fmaf(wj, t[k], v[k]);
+        }
+    } else {
+        ldb<V>(x, p.table + (size_t)p.tokens[src] * p.dim + i);
+    }
+    if (SRC != 2) {
+        if (p.scale) {
+            float s[V];
+            ldb<V>(s, p.scale + i);
+#pragma unroll
+            for (int k = 0; k < V; k++) x[k] = fmaf(s[k], v[k], x[k]);
+        } else {
+#pragma unroll
+            for (int k = 0; k < V; k++) x[k] += v[k];
+        }
+    }
+    if (!p.row_idx) stf<V>(p.res + (size_t)r * p.dim + i, x);
+    if (!p.w) return;
+    const float al = bf16_bits_to_f32(*p.alpha);
+    float w[V], b[V], h[V];
+    ldb<V>(w, p.w + i), ldb<V>(b, p.b + i);
+#pragma unroll
+    for (int k = 0; k < V; k++) h[k] = fmaf(tanhf(al * x[k]), w[k], b[k]);
+    if (!p.mu) {
+        st_act<TO, V>((TO*)p.out + (size_t)r * p.dim + i, h);
+        return;
+    }
+    float* tail = p.tail + (size_t)p.slot[r] * p.tail_stride + i;
+    float d[V];
+    ldf<V>(d, tail);
+    stf<V>(tail, h);
+    const bool first = p.pos[r] == 0;
+#pragma unroll
+    for (int k = 0; k < V; k++) d[k] = (first ? 0.f : d[k]) - h[k];
+    for (int q = 0; q < p.n_mix; q++) {
+        float m[V], o[V];
+        ldb<V>(m, p.mu + (size_t)q * p.dim + i);
+#pragma unroll
+        for (int k = 0; k < V; k++) o[k] = fmaf(d[k], m[k], h[k]);
+        st_act<TO, V>((TO*)p.out + (size_t)q * p.plane + (size_t)r * p.dim + i, o);
+    }
+}
+// The mixes of a panel (rows seq * T + t of the finished stream): a thread walks kShiftRows tokens of its entries and keeps the last h.  The
+// block row of t = 0 reads the tail and leaves the sequence's last h there, so nobody else touches it.
+template <typename TO, int V>
+__global__ void __launch_bounds__(128) kf_dyt_mix_kernel(DytArgs p) {
+    const int i = (blockIdx.x * blockDim.x + threadIdx.x) * V, seq = blockIdx.z, T = p.T;
+    if (i >= p.dim) return;
+    const int t0 = blockIdx.y * kShiftRows, t1 = min(T, t0 + kShiftRows);
+    const float al = bf16_bits_to_f32(*p.alpha);
+    float w[V], b[V], prev[V];
+    ldb<V>(w, p.w + i), ldb<V>(b, p.b + i);
+    const float* xs = p.res + (size_t)seq * T * p.dim + i;
+    auto norm = [&](float (&h)[V], int t) {
+        ldf<V>(h, xs + (size_t)t * p.dim);
+#pragma unroll
+        for (int k = 0; k < V; k++) h[k] = fmaf(tanhf(al * h[k]), w[k], b[k]);
+    };
+    if (t0 == 0) {
+        float* tl = p.tail + (size_t)p.slot[(size_t)seq * T] * p.tail_stride + i;
+        float last[V];
+        ldf<V>(prev, tl);
+        norm(last, T - 1);
+        stf<V>(tl, last);
+    } else {
+        norm(prev, t0 - 1);
+    }
+    for (int t = t0; t < t1; t++) {
+        float h[V], d[V];
+        norm(h, t);
+        const bool first = p.pos[(size_t)seq * T + t] == 0;
+#pragma unroll
+        for (int k = 0; k < V; k++) d[k] = (first ? 0.f : prev[k]) - h[k], prev[k] = h[k];
+        for (int q = 0; q < p.n_mix; q++) {
+            float m[V], o[V];
+            ldb<V>(m, p.mu + (size_t)q * p.dim + i);
+#pragma unroll
+            for (int k = 0; k < V; k++) o[k] = fmaf(d[k], m[k], h[k]);
+            st_act<TO, V>((TO*)p.out + (size_t)q * p.plane + ((size_t)seq * T + t) * p.dim + i, o);
+        }
+    }
+}
+bool dyt_args(DytArgs& p, const kf_dyt_step* s) {
+    p.res = s->res, p.dim = s->dim, p.scale = (const uint16_t*)s->scale_bf16, p.w = (const uint16_t*)s->w_bf16, p.b = (const uint16_t*)s->b_bf16;
+    p.alpha = (const uint16_t*)s->alpha_bf16, p.out = s->out, p.row_idx = s->row_idx, p.mu = (const uint16_t*)s->mu_bf16, p.n_mix = s->n_mix, p.plane = s->plane;
+    p.tail = s->tail, p.tail_stride = s->tail_stride, p.pos = s->pos, p.slot = s->slot;
+    if (!s->res || s->rows < 1 || s->rows > 65535 || s->dim < 1 || (s->w_bf16 && (!s->b_bf16 || !s->alpha_bf16 || !s->out))) return false;
+    return !s->mu_bf16 || (s->w_bf16 && s->n_mix >= 1 && s->plane >= (size_t)s->rows * s->dim && s->tail && s->tail_stride >= (size_t)s->dim && s->pos && s->slot && !s->row_idx);
+}
+// four entries per access: row length and every row's address allow it
+bool dyt_vec(const DytArgs& p) {
+    const uintptr_t at16 = (uintptr_t)p.res | (uintptr_t)p.out | (uintptr_t)p.a | (uintptr_t)p.y | (uintptr_t)p.tail | (uintptr_t)p.pass;
+    const uintptr_t at8  = (uintptr_t)p.scale | (uintptr_t)p.w | (uintptr_t)p.b | (uintptr_t)p.mu | (uintptr_t)p.table;
+    return p.dim % 4 == 0 && p.lda % 4 == 0 && p.plane % 4 == 0 && p.tail_stride % 4 == 0 && at16 % 16 == 0 && at8 % 8 == 0;
+}
+template <int SRC>
+int launch_dyt(kf_ctx* ctx, const DytArgs& p, int out_f32, int rows) {
+    const int v = dyt_vec(p) ? 4 : 1;
+    const dim3 grid((p.dim + 128 * v - 1) / (128 * v), rows);
+#define KF_DYT(T, V) kf_dyt_step_kernel<SRC, T, V><<<grid, 128, 0, ctx->stream>>>(p)
+    if (out_f32) v == 4 ? KF_DYT(float, 4) : KF_DYT(float, 1);
+    else v == 4 ? KF_DYT(uint16_t, 4) : KF_DYT(uint16_t, 1);
+#undef KF_DYT
+    KF_LAUNCH_CHECK(ctx);
+    return KF_OK;
+}
 // out = g' * sigmoid(alpha * g') * (u' + shift),  g' = min(g, limit), u' = clamp(u, -limit, limit)  (limit <= 0: not clamped)
 template <typename TO>
 __global__ void kf_glu_clamped_kernel(TO* __restrict__ out, int ldo, const float* __restrict__ g, int ldg, const float* __restrict__ u, int ldu, int cols,
@@ -361,52 +534,77 @@ __global__ void kf_f32_to_bf16_kernel(uint16_t* __restrict__ out, const float* _
 // kind 1: scores s = sigmoid(logit); the choice runs over s + bias; the experts form `groups` equal contiguous groups, a group is ranked
 // by the sum of its top-2 choice values and only the `keep` best groups can be chosen from; weights = scale * s of the chosen, not
 // renormalised.
+// kind 2: scores s = softmax(logits) over all outputs; choice over s + bias inside the `keep` best groups as in kind 1, but a group is ranked by
+// its LARGEST choice value; weights = s of the chosen over (their sum + 1e-20).
+// The last `pass` outputs of the router (kind 2) are no experts: an entry that goes to one takes no slot (entry_slot -1), the combination reads
+// the sublayer's input for it.
 struct RouteMode {
     int kind, groups, keep;
     float scale;
+    int pass;
 };
-// one warp routes one token in kind 1.  taken: the token's chosen experts so far (shared or global memory, written by lane 0).
+constexpr int kRouteGroups = 64;
+// one warp routes one token in kinds 1 and 2.  taken: the token's chosen experts so far (shared or global memory, written by lane 0).
 __device__ __forceinline__ void route_grouped_warp(int* taken, int32_t* idx, float* __restrict__ wgt, const float* __restrict__ lg,
                                                    const uint16_t* __restrict__ bias, int E, int top, const RouteMode md, int lane) {
     const int per = E / md.groups;
-    // lane g keeps the rank value of group g (groups <= 32): the top-2 choice values of the group, found by all lanes together
-    float gscore = -INFINITY;
-    for (int g = 0; g < md.groups; g++) {
-        float a = -INFINITY, b = -INFINITY;  // largest, second largest of this lane's share
-        for (int e = g * per + lane; e < (g + 1) * per; e += 32) {
-            const float v = sigmoid_f(lg[e]) + (bias ? bf16_bits_to_f32(bias[e]) : 0.f);
-            if (v > a) b = a, a = v;
-            else if (v > b) b = v;
-        }
-#pragma unroll
-        for (int o = 16; o > 0; o >>= 1) {
-            const float oa = __shfl_xor_sync(0xffffffffu, a, o), ob = __shfl_xor_sync(0xffffffffu, b, o);
-            const float hi = fmaxf(a, oa), lo = fmaxf(fminf(a, oa), fmaxf(b, ob));
-            a = hi, b = lo;
-        }
-        if (lane == g) gscore = per > 1 ? a + b : a;
+    float mx = 0.f, inv = 1.f;
+    if (md.kind == 2) {
+        mx = -INFINITY;
+        for (int e = lane; e < E; e += 32) mx = fmaxf(mx, lg[e]);
+        mx = warp_max(mx);
+        float d = 0.f;
+        for (int e = lane; e < E; e += 32) d += expf(lg[e] - mx);
+        inv = 1.f / warp_sum(d);
     }
-    unsigned kept = 0;
-    for (int r = 0; r < md.keep; r++) {
-        float best = (lane < md.groups && !((kept >> lane) & 1u)) ? gscore : -INFINITY;
-        int bi     = (lane < md.groups && !((kept >> lane) & 1u)) ? lane : 0x7fffffff;
+    auto score  = [&](int e) { return md.kind == 2 ? expf(lg[e] - mx) * inv : sigmoid_f(lg[e]); };
+    auto choice = [&](int e) { return score(e) + (bias ? bf16_bits_to_f32(bias[e]) : 0.f); };
+    unsigned long long kept = 0;
+    if (md.keep >= md.groups) {
+        kept = ~0ull;
+    } else {
+        // lane g & 31 keeps the rank values of groups g and g + 32, found by all lanes together
+        float gs0 = -INFINITY, gs1 = -INFINITY;
+        for (int g = 0; g < md.groups; g++) {
+            float a = -INFINITY, b = -INFINITY;  // largest, second largest of this lane's share
+            for (int e = g * per + lane; e < (g + 1) * per; e += 32) {
+                const float v = choice(e);
+                if (v > a) b = a, a = v;
+                else if (v > b) b = v;
+            }
 #pragma unroll
-        for (int o = 16; o > 0; o >>= 1) {
-            const float ob = __shfl_xor_sync(0xffffffffu, best, o);
-            const int oi   = __shfl_xor_sync(0xffffffffu, bi, o);
-            if (oi != 0x7fffffff && (bi == 0x7fffffff || ob > best || (ob == best && oi < bi))) best = ob, bi = oi;
+            for (int o = 16; o > 0; o >>= 1) {
+                const float oa = __shfl_xor_sync(0xffffffffu, a, o), ob = __shfl_xor_sync(0xffffffffu, b, o);
+                const float hi = fmaxf(a, oa), lo = fmaxf(fminf(a, oa), fmaxf(b, ob));
+                a = hi, b = lo;
+            }
+            const float rank = (md.kind == 1 && per > 1) ? a + b : a;
+            if (lane == (g & 31)) (g < 32 ? gs0 : gs1) = rank;
         }
-        if (bi != 0x7fffffff) kept |= 1u << bi;
+        for (int r = 0; r < md.keep; r++) {
+            float best = -INFINITY;
+            int bi     = 0x7fffffff;
+            if (lane < md.groups && !((kept >> lane) & 1ull)) best = gs0, bi = lane;
+            if (lane + 32 < md.groups && !((kept >> (lane + 32)) & 1ull) && (bi == 0x7fffffff || gs1 > best)) best = gs1, bi = lane + 32;
+#pragma unroll
+            for (int o = 16; o > 0; o >>= 1) {
+                const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+                const int oi   = __shfl_xor_sync(0xffffffffu, bi, o);
+                if (oi != 0x7fffffff && (bi == 0x7fffffff || ob > best || (ob == best && oi < bi))) best = ob, bi = oi;
+            }
+            if (bi != 0x7fffffff) kept |= 1ull << bi;
+        }
     }
+    float sum = 0.f;
     for (int j = 0; j < top; j++) {
         float best = -INFINITY;
         int bi     = 0x7fffffff;
         for (int e = lane; e < E; e += 32) {
-            if (!((kept >> (e / per)) & 1u)) continue;
+            if (!((kept >> min(63, e / per)) & 1ull)) continue;
             bool was = false;
             for (int q = 0; q < j; q++) was = was || taken[q] == e;
             if (was) continue;
-            const float v = sigmoid_f(lg[e]) + (bias ? bf16_bits_to_f32(bias[e]) : 0.f);
+            const float v = choice(e);
             if (bi == 0x7fffffff || v > best || (v == best && e < bi)) best = v, bi = e;
         }
 #pragma unroll
@@ -415,9 +613,15 @@ __device__ __forceinline__ void route_grouped_warp(int* taken, int32_t* idx, flo
             const int oi   = __shfl_xor_sync(0xffffffffu, bi, o);
             if (oi != 0x7fffffff && (bi == 0x7fffffff || ob > best || (ob == best && oi < bi))) best = ob, bi = oi;
         }
-        if (lane == 0) taken[j] = bi, idx[j] = bi, wgt[j] = md.scale * sigmoid_f(lg[bi]);
+        if (lane == 0) {
+            const float sc = score(bi);
+            sum += sc;
+            taken[j] = bi, idx[j] = bi, wgt[j] = md.kind == 2 ? sc : md.scale * sc;
+        }
         __syncwarp();
     }
+    if (md.kind == 2 && lane == 0)
+        for (int j = 0; j < top; j++) wgt[j] /= sum + 1e-20f;
 }
 // one warp per token: `top` rounds of arg-max over the E router logits (+ bias), ties to the lower index; weights = softmax over the
 // chosen logits only, or (full) the chosen entries of the softmax over ALL experts, not renormalised.  All in fp32.
@@ -426,7 +630,7 @@ __global__ void __launch_bounds__(128) kf_moe_route_kernel(int32_t* __restrict__
     const int m = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
     if (m >= M) return;
     const float* lg = logits + (size_t)m * ldl;
-    if (md.kind == 1) {
+    if (md.kind) {
         route_grouped_warp(idx + (size_t)m * top, idx + (size_t)m * top, wgt + (size_t)m * top, lg, bias, E, top, md, lane);
         return;
     }
@@ -463,7 +667,8 @@ __global__ void __launch_bounds__(128) kf_moe_route_kernel(int32_t* __restrict__
     }
 }
 // The dispatch tables of a few entries by ONE block of 256 threads: entry i = (token i / top, choice i % top) goes to expert sidx[i]; thread i
-// ranks its entry among the earlier ones of its expert, the lanes of warp 0 count one expert each and scan the counts.
+// ranks its entry among the earlier ones of its expert, the lanes of warp 0 count one expert each and scan the counts.  Entries of outputs
+// beyond the E experts take no slot; the slots that stay free are marked with group -1.
 constexpr int kRouteSmall = 256;
 __device__ __forceinline__ void dispatch_small(const int* sidx, int* srank, int n, int E, int top, int32_t* offsets, int32_t* entry_slot, int32_t* slot_row,
                                                int32_t* slot_group) {
@@ -494,7 +699,13 @@ __device__ __forceinline__ void dispatch_small(const int* sidx, int* srank, int 
     }
     __syncthreads();
     for (int i = threadIdx.x; i < n; i += blockDim.x) {
-        const int e = sidx[i], sl = offsets[e] + srank[i];
+        if (i >= offsets[E]) slot_row[i] = 0, slot_group[i] = -1;
+        const int e = sidx[i];
+        if (e >= E) {
+            entry_slot[i] = -1;
+            continue;
+        }
+        const int sl = offsets[e] + srank[i];
         entry_slot[i] = sl, slot_row[sl] = i / top, slot_group[sl] = e;
     }
 }
@@ -508,7 +719,7 @@ __global__ void __launch_bounds__(256) kf_moe_route_small_kernel(int32_t* __rest
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, n = M * top;
     for (int m = warp; m < M; m += 8) {
         const float* lg = logits + (size_t)m * ldl;
-        if (md.kind == 1) {
+        if (md.kind) {
             route_grouped_warp(sidx + m * top, idx + (size_t)m * top, wgt + (size_t)m * top, lg, bias, E, top, md, lane);
             continue;
         }
@@ -542,7 +753,7 @@ __global__ void __launch_bounds__(256) kf_moe_route_small_kernel(int32_t* __rest
         }
         for (int j = lane; j < top; j += 32) wgt[(size_t)m * top + j] /= den;
     }
-    dispatch_small(sidx, srank, n, E, top, offsets, entry_slot, slot_row, slot_group);
+    dispatch_small(sidx, srank, n, E - md.pass, top, offsets, entry_slot, slot_row, slot_group);
 }
 // one block per expert: the entries (token, choice) routed to it, ranked in entry order (ballot + popc compaction)
 __device__ __forceinline__ void rank_expert(int32_t* rank, int32_t* count, const int32_t* idx, int n, int e) {
@@ -582,10 +793,17 @@ __global__ void kf_moe_offsets_kernel(int32_t* __restrict__ offsets, const int32
     }
 }
 __global__ void kf_moe_slots_kernel(int32_t* __restrict__ entry_slot, int32_t* __restrict__ slot_row, int32_t* __restrict__ slot_group,
-                                    const int32_t* __restrict__ idx, const int32_t* __restrict__ rank, const int32_t* __restrict__ offsets, int n, int top) {
+                                    const int32_t* __restrict__ idx, const int32_t* __restrict__ rank, const int32_t* __restrict__ offsets, int n, int top,
+                                    int E) {
     const int i = blockIdx.x * blockDim.x + threadIdx.x;
     if (i >= n) return;
-    const int e = idx[i], s = offsets[e] + rank[i];
+    if (i >= offsets[E]) slot_row[i] = 0, slot_group[i] = -1;  // no entry has this slot
+    const int e = idx[i];
+    if (e >= E) {
+        entry_slot[i] = -1;
+        return;
+    }
+    const int s = offsets[e] + rank[i];
     entry_slot[i] = s, slot_row[s] = i / top, slot_group[s] = e;
 }
 // Routing from a table of token ids: row tokens[m] names the token's `top` experts, each with weight 1 / top -- no logits.  It depends on
@@ -838,6 +1056,46 @@ extern "C" int kf_glu_clamped(kf_ctx* ctx, void* out, int out_f32, int ldo, cons
     KF_LAUNCH_CHECK(ctx);
     return KF_OK;
 }
+// Steps of a stack with the norm n(x) = tanh(alpha x) w + b (see kf_dyt_step): x = res + scale * a, out = n(x) or the token mixes of n(x).
+extern "C" int kf_dyt_residual(kf_ctx* ctx, const kf_dyt_step* s, const float* a, int lda) {
+    if (!ctx || !s) return KF_ERR_BAD_ARG;
+    DytArgs p = {};
+    KF_REQUIRE(ctx, dyt_args(p, s) && (!a || lda >= s->dim), "rows, norm, mixes");
+    p.a = a, p.lda = lda;
+    return launch_dyt<0>(ctx, p, s->out_f32, s->rows);
+}
+// The same over a token's experts: the added row is sum_j wgt[m][j] * y_slots[entry_slot[m][j]]; an entry without a slot (-1) stands for row m of
+// `pass` ([rows][dim] in the activation type), which may be the buffer that out writes.
+extern "C" int kf_dyt_experts(kf_ctx* ctx, const kf_dyt_step* s, const float* y_slots, const int32_t* entry_slot, const float* wgt, const void* pass, int top) {
+    if (!ctx || !s || !y_slots || !entry_slot || !wgt || !pass) return KF_ERR_BAD_ARG;
+    DytArgs p = {};
+    KF_REQUIRE(ctx, dyt_args(p, s) && top >= 1 && !(s->row_idx && pass == s->out), "rows, norm, mixes");
+    p.y = y_slots, p.entry_slot = entry_slot, p.wgt = wgt, p.pass = pass, p.top = top;
+    return launch_dyt<1>(ctx, p, s->out_f32, s->rows);
+}
+// The start of a stream: res[m] = W[token[m]], out as above.
+extern "C" int kf_dyt_embed(kf_ctx* ctx, const kf_dyt_step* s, const kf_tensor_desc* table, const int32_t* tokens) {
+    if (!ctx || !s || !table || !table->data_dev || !tokens) return KF_ERR_BAD_ARG;
+    DytArgs p = {};
+    KF_REQUIRE(ctx, dyt_args(p, s) && !s->row_idx && table->type == KF_T_BF16 && table->cols == s->dim, "bf16 table of the stream's width");
+    p.table = (const uint16_t*)table->data_dev, p.tokens = tokens;
+    return launch_dyt<2>(ctx, p, s->out_f32, s->rows);
+}
+// The token mixes of n(res) for nseq sequences of T consecutive tokens each (res is only read; rows = nseq * T).
+extern "C" int kf_dyt_token_mix(kf_ctx* ctx, const kf_dyt_step* s, int nseq, int T) {
+    if (!ctx || !s) return KF_ERR_BAD_ARG;
+    DytArgs p = {};
+    KF_REQUIRE(ctx, dyt_args(p, s) && s->mu_bf16 && nseq >= 1 && nseq <= 65535 && T >= 1 && s->rows == nseq * T, "rows, norm, mixes");
+    p.T = T;
+    const int v = dyt_vec(p) ? 4 : 1;
+    const dim3 grid((p.dim + 128 * v - 1) / (128 * v), (T + kShiftRows - 1) / kShiftRows, nseq);
+#define KF_DYM(TY, V) kf_dyt_mix_kernel<TY, V><<<grid, 128, 0, ctx->stream>>>(p)
+    if (s->out_f32) v == 4 ? KF_DYM(float, 4) : KF_DYM(float, 1);
+    else v == 4 ? KF_DYM(uint16_t, 4) : KF_DYM(uint16_t, 1);
+#undef KF_DYM
+    KF_LAUNCH_CHECK(ctx);
+    return KF_OK;
+}
 extern "C" int kf_scale_f32(kf_ctx* ctx, float* x, size_t n, float s) {
     if (!ctx || !x) return KF_ERR_BAD_ARG;
     if (!n || s == 1.f) return KF_OK;
@@ -870,29 +1128,45 @@ static int moe_route_impl(kf_ctx* ctx, int32_t* idx, float* wgt, int32_t* offset
     int32_t *rank = work, *count = work + n;
     kf_moe_route_kernel<<<(M + 3) / 4, 128, 0, ctx->stream>>>(idx, wgt, logits, ldl, (const uint16_t*)bias_bf16, M, E, top, full_softmax, md);
     KF_LAUNCH_CHECK(ctx);
-    kf_moe_rank_kernel<<<E, 256, 0, ctx->stream>>>(rank, count, idx, n);
+    const int X = E - md.pass;
+    kf_moe_rank_kernel<<<X, 256, 0, ctx->stream>>>(rank, count, idx, n);
     KF_LAUNCH_CHECK(ctx);
-    kf_moe_offsets_kernel<<<1, 32, 0, ctx->stream>>>(offsets, count, E);
+    kf_moe_offsets_kernel<<<1, 32, 0, ctx->stream>>>(offsets, count, X);
     KF_LAUNCH_CHECK(ctx);
-    kf_moe_slots_kernel<<<(n + 255) / 256, 256, 0, ctx->stream>>>(entry_slot, slot_row, slot_group, idx, rank, offsets, n, top);
+    kf_moe_slots_kernel<<<(n + 255) / 256, 256, 0, ctx->stream>>>(entry_slot, slot_row, slot_group, idx, rank, offsets, n, top, X);
     KF_LAUNCH_CHECK(ctx);
     return KF_OK;
 }
 extern "C" int kf_moe_route_ex(kf_ctx* ctx, int32_t* idx, float* wgt, int32_t* offsets, int32_t* entry_slot, int32_t* slot_row, int32_t* slot_group,
                                int32_t* work, const float* logits, int ldl, const void* bias_bf16, int M, int E, int top, int full_softmax) {
-    const RouteMode md = {0, 1, 1, 1.f};
+    const RouteMode md = {0, 1, 1, 1.f, 0};
     return moe_route_impl(ctx, idx, wgt, offsets, entry_slot, slot_row, slot_group, work, logits, ldl, bias_bf16, M, E, top, full_softmax, md);
 }
 // The same tables from sigmoid scores: the choice runs over sigmoid(logit) + choice_bias (bf16 [E] or NULL) inside the `keep` best of
-// `groups` equal contiguous groups of experts (a group ranks by the sum of its top-2 choice values; groups <= 32, groups 1: no
+// `groups` equal contiguous groups of experts (a group ranks by the sum of its top-2 choice values; groups <= 64, groups 1: no
 // grouping); weights = scale * sigmoid(logit) of the chosen experts, not renormalised.  top <= keep * (E / groups).
 extern "C" int kf_moe_route_grouped(kf_ctx* ctx, int32_t* idx, float* wgt, int32_t* offsets, int32_t* entry_slot, int32_t* slot_row, int32_t* slot_group,
                                     int32_t* work, const float* logits, int ldl, const void* choice_bias_bf16, int M, int E, int top, int groups, int keep,
                                     float scale) {
     if (!ctx) return KF_ERR_BAD_ARG;
-    KF_REQUIRE(ctx, groups >= 1 && groups <= 32 && E >= 1 && E % groups == 0 && keep >= 1 && keep <= groups && top >= 1 && top <= keep * (E / groups),
-               "groups <= 32 divide the experts; 1 <= keep <= groups; top <= keep * experts / groups");
-    const RouteMode md = {1, groups, keep, scale};
+    KF_REQUIRE(ctx, groups >= 1 && groups <= kRouteGroups && E >= 1 && E % groups == 0 && keep >= 1 && keep <= groups && top >= 1 && top <= keep * (E / groups),
+               "groups <= 64 divide the experts; 1 <= keep <= groups; top <= keep * experts / groups");
+    const RouteMode md = {1, groups, keep, scale, 0};
+    return moe_route_impl(ctx, idx, wgt, offsets, entry_slot, slot_row, slot_group, work, logits, ldl, choice_bias_bf16, M, E, top, 0, md);
+}
+// The same tables from softmax scores over experts + pass outputs (logits [M][ldl >= experts + pass]): the choice runs over s + choice_bias
+// inside the `keep` best of `groups` equal contiguous groups of the outputs (a group ranks by its largest choice value; groups <= 64);
+// weights = s of the chosen over (their sum + 1e-20).  The last `pass` outputs are no experts: their entries get entry_slot -1 and no slot,
+// slots that stay unused get slot_group -1.
+extern "C" int kf_moe_route_softmax_grouped(kf_ctx* ctx, int32_t* idx, float* wgt, int32_t* offsets, int32_t* entry_slot, int32_t* slot_row, int32_t* slot_group,
+                                            int32_t* work, const float* logits, int ldl, const void* choice_bias_bf16, int M, int experts, int pass, int top,
+                                            int groups, int keep) {
+    if (!ctx) return KF_ERR_BAD_ARG;
+    const int E = experts + pass;
+    KF_REQUIRE(ctx, experts >= 1 && pass >= 0 && groups >= 1 && groups <= kRouteGroups && E % groups == 0 && keep >= 1 && keep <= groups && top >= 1 &&
+                        top <= keep * (E / groups),
+               "groups <= 64 divide the outputs; 1 <= keep <= groups; top <= keep * outputs / groups");
+    const RouteMode md = {2, groups, keep, 1.f, pass};
     return moe_route_impl(ctx, idx, wgt, offsets, entry_slot, slot_row, slot_group, work, logits, ldl, choice_bias_bf16, M, E, top, 0, md);
 }
 extern "C" int kf_moe_route(kf_ctx* ctx, int32_t* idx, float* wgt, int32_t* offsets, int32_t* entry_slot, int32_t* slot_row, int32_t* slot_group,

@@ -23,7 +23,8 @@ namespace koifish {
 struct MIXER_CARD {
     std::string type;  // "mamba2" (state-space) | "latent_attention" | "channel_delta" | "gla" | "parallel" (attention beside a gated LRU) |
                        // "mingru" (channel-wise gated recurrence) | "attention" (Fazolorn: sigmoid-weighted, inside blocks of positions;
-                       // Gadilix: softmax over a sliding window and pooled blocks behind it)
+                       // Gadilix: softmax over a sliding window and pooled blocks behind it; Zadinex: softmax with a sink, values blended
+                       // over the layers) | "wkv" (time mixing with a bonus)
     // state-space mixer: heads x vdim inner channels, state rows per head, B/C groups, gated-norm groups, convolution taps
     int heads = 0, vdim = 0, state = 0, groups = 1, norm_groups = 1, conv = 1;
     // latent attention: per head `dim` plain + `rot_dim` rotated query/key entries, values of vdim, latent rank; rotation on the first
@@ -52,6 +53,8 @@ struct MIXER_CARD {
     int block = 0;
     // beside the window of `window` positions one mean key and value for every block of `pool` positions that lies wholly before it (0: none)
     int pool = 0;
+    // the layer's values are blended with those of the first layer that says so
+    bool v_mix = false;
     // channel-wise gated recurrence (minGRU): channels of the state
     int width = 0;
     // two mixers side by side that read the same input (Sedotar's "parallel"): this card is the left one, `right` the other; the result is
@@ -70,6 +73,12 @@ struct MOE_CARD {
     bool sigmoid_route = false;
     int groups = 1, keep = 1;
     float route_scale = 1.f;
+    // routing from softmax scores over experts + `pass` pass-through outputs: selection over score + a learned correction inside the `keep` best
+    // of `groups` groups of neighbouring outputs (ranked by their largest), weights renormalised over the chosen
+    bool softmax_groups = false;
+    int pass = 0;
+    // experts of the form g sigmoid(glu_alpha g) (u + glu_shift), clamped by `limit` when positive (glu_alpha 0: silu(g) u)
+    float glu_alpha = 0.f, glu_shift = 0.f;
     bool table_route = false;  // no router: a table [vocab][top] names the experts of every token id, each with weight 1 / top
 };
 struct LAYER_CARD {
@@ -221,6 +230,7 @@ const ARCH_ENTRY* KivoraxArch();  // Kivorax.cpp
 const ARCH_ENTRY* SedotarArch();  // Sedotar.cpp
 const ARCH_ENTRY* FazolornArch(); // Fazolorn.cpp
 const ARCH_ENTRY* GadilixArch();  // Gadilix.cpp
+const ARCH_ENTRY* ZadinexArch();  // Zadinex.cpp
 
 // ---- the model ------------------------------------------------------------------------------------------------------------
 struct Fish {

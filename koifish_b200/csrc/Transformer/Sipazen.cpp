@@ -366,7 +366,11 @@ int MoE::Experts(int M, const int32_t* offsets, const int32_t* slot_row, const i
     const int E = f.config.n_embd, X = card.experts, top = card.top;
     const int ak = f.config.compute_f32 ? 1 : 0;
     const void* const* tb = (const void* const*)tables;
-    KF_TRY(kf_linear_grouped(f.ctx, s.h1, card.ff, tb, tb + X, X, card.ff, E, s.hact, ak, E, offsets, slot_group, slot_row, M * top));
+    if (card.glu_alpha > 0.f)
+        KF_TRY(kf_linear_grouped_glu(f.ctx, s.h1, card.ff, tb, tb + X, X, card.ff, E, s.hact, ak, E, offsets, slot_group, slot_row, M * top, card.limit, card.glu_alpha,
+                                     card.glu_shift));
+    else
+        KF_TRY(kf_linear_grouped(f.ctx, s.h1, card.ff, tb, tb + X, X, card.ff, E, s.hact, ak, E, offsets, slot_group, slot_row, M * top));
     KF_TRY(kf_linear_grouped(f.ctx, s.yslots, E, tb + 2 * X, nullptr, X, E, card.ff, s.h1, ak, card.ff, offsets, slot_group, nullptr, M * top));
     if (card.shared_ff > 0) {
         kf_tensor_desc dg = sh_gate->Desc(), du = sh_up->Desc();
@@ -376,17 +380,29 @@ int MoE::Experts(int M, const int32_t* offsets, const int32_t* slot_row, const i
     return KF_OK;
 }
 
-int MoE::cuInfer(int M, const float* u, int ldu, int off_router, int off_sg, float* into_residual) {
+int MoE::Route(int M, const float* u, int ldu, int off_router) {
     Fish& f = *hFish;
     std::string* hFishErr = &f.error;
     HybridScratch& s = *f.hscratch;
-    const int E = f.config.n_embd, X = card.experts, top = card.top;
+    const int X = card.experts, top = card.top;
     const void* rb = router_b ? router_b->data : nullptr;
-    if (card.sigmoid_route)
+    if (card.softmax_groups)
+        KF_TRY(kf_moe_route_softmax_grouped(f.ctx, s.idx, s.wgt, s.offsets, s.entry_slot, s.slot_row, s.slot_group, s.work, u + off_router, ldu, rb, M, X, card.pass, top,
+                                            card.groups, card.keep));
+    else if (card.sigmoid_route)
         KF_TRY(kf_moe_route_grouped(f.ctx, s.idx, s.wgt, s.offsets, s.entry_slot, s.slot_row, s.slot_group, s.work, u + off_router, ldu, rb, M, X, top, card.groups,
                                     card.keep, card.route_scale));
     else
         KF_TRY(kf_moe_route(f.ctx, s.idx, s.wgt, s.offsets, s.entry_slot, s.slot_row, s.slot_group, s.work, u + off_router, ldu, rb, M, X, top));
+    return KF_OK;
+}
+
+int MoE::cuInfer(int M, const float* u, int ldu, int off_router, int off_sg, float* into_residual) {
+    Fish& f = *hFish;
+    std::string* hFishErr = &f.error;
+    HybridScratch& s = *f.hscratch;
+    const int E = f.config.n_embd, top = card.top;
+    KF_TRY(Route(M, u, ldu, off_router));
     KF_TRY(Experts(M, s.offsets, s.slot_row, s.slot_group));
     const bool sh = card.shared_ff > 0;
     KF_TRY(kf_moe_combine_ex(f.ctx, into_residual ? into_residual : s.sub, s.yslots, s.entry_slot, s.wgt, sh ? s.shared : nullptr, sh ? u + off_sg : nullptr, ldu,

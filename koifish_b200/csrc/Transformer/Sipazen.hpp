@@ -28,6 +28,7 @@ struct HybridScratch {  // device buffers shared by all layers, sized for max_to
     // stacks with low-rank projections, a per-layer token input, a depth-weighted residual, a gated LRU
     void* mid = nullptr;         // second-stage matmul inputs (low-rank middles, token-gated side input), activation type
     float* hist = nullptr;       // [layers + 1][T][E] results of the embedding and of every layer
+    float* vfirst = nullptr;     // [T][kv heads x vdim] values of the first layer that blends its values
     float* lru_work = nullptr;   // [2][T][widest LRU]: decay and input term of every token
 };
 
@@ -77,6 +78,7 @@ struct MoE : GeNeuron {
     int Experts(int M, const int32_t* offsets, const int32_t* slot_row, const int32_t* slot_group);
     // into_residual: the weighted sum of the experts is added to that buffer instead of being written to the sublayer result
     int cuInfer(int M, const float* u, int ldu, int off_router, int off_sg, float* into_residual = nullptr);
+    int Route(int M, const float* u, int ldu, int off_router);  // logits -> the scratch's dispatch tables and weights
 };
 struct HybridBlock : GeNeuron {
     int layer = 0;
