@@ -1,10 +1,11 @@
-"""Prefill and decode throughput of a hybrid stack (bench.py --compare-arch sipazen | kivorax | sedotar | fazolorn | gadilix) beside the closest existing
+"""Prefill and decode throughput of a hybrid stack (bench.py --compare-arch sipazen | kivorax | sedotar | fazolorn | gadilix | zadinex) beside the closest existing
 models at equal width, depth and active feed-forward width: Sipazen beside Qwen3; Kivorax beside Sipazen (the other recurrence + attention +
 experts stack of this runtime) and Qwen3; Sedotar (sliding-window attention beside a delta rule, dense feed-forward) beside Kivorax with
 dense feed-forwards (delta-rule layers and attention layers alternating) and Qwen3; Fazolorn (minGRU, sigmoid block attention and latent
 attention layers with routed experts) beside Sipazen (state-space and latent attention layers with routed experts) and Qwen3; Gadilix
 (windowed attention beside pooled blocks, experts by token id beside a shared one) beside Sipazen (the same experts and shared expert behind a
-router), Sedotar (the same attention heads and window, dense feed-forward) and Qwen3.  All bf16 with random weights.  One JSON line per (model, size).
+router), Sedotar (the same attention heads and window, dense feed-forward) and Qwen3; Zadinex (time-mixing and attention layers with routed
+experts) beside Kivorax (delta-rule, gated linear attention and attention layers with the same experts) and Qwen3.  All bf16 with random weights.  One JSON line per (model, size).
 
     prefill: a prompt of --prompt tokens through the model's own step function in panels, timed with CUDA events after 3 warm-up prompts
     decode : the device-resident greedy loop (one CUDA-graph replay per token) at context --prompt, after W warm-up tokens
@@ -112,6 +113,27 @@ def gadilix_config(p):
     return {"architecture": "Gadilix", "vocab": p["vocab"], "width": w, "residual_mult": 0.5, "norm": {"eps": 1e-5}, "layers": [ly] * len(p["pattern"])}
 
 
+def zadinex_config(p):
+    """Kivorax's order of layers: time mixing (heads of 64 over the model width, a decay of the preset's low rank) where that stack has a delta rule
+    or gated linear attention, attention (head size 128, 4 query heads per kv head, half of each head rotated, blended values) where it has
+    attention beside an LRU; the first feed-forward dense, the others the preset's experts and top plus an eighth as many pass-through outputs,
+    in 3 groups of which 2 are kept"""
+    w, m, k = p["width"], p["moe"], p["kvx"]
+    heads = w // 128
+    outs = m["experts"] // 8
+    layers = []
+    for i, ch in enumerate(k["pattern"]):
+        if ch == "p":
+            typ, mixer = "attention", dict(heads=heads, kv_heads=max(1, heads // 4), dim=128, vdim=128, scale=128 ** -0.5, v_mix=True, rot=dict(base=1e6, dims=64))
+        else:
+            typ, mixer = "wkv", dict(heads=w // 64, dim=64, w_rank=k["rank"])
+        mlp = {"kind": "dense", "ff": m["top"] * m["ff"]} if i == 0 else \
+            {"kind": "moe", "expert": {"ff": m["ff"], "limit": 7.0},
+             "router": {"experts": m["experts"], "identity": outs, "top": m["top"], "groups": {"count": 3, "keep": 2}}}
+        layers.append({"type": typ, "mixer": mixer, "mlp": mlp})
+    return {"architecture": "Zadinex", "vocab": p["vocab"], "width": w, "norm": {"eps": 1e-5}, "layers": layers}
+
+
 def kivorax_dense_config(p):
     """Kivorax at the size of sedotar_config: delta-rule layers and attention (+ LRU) layers alternating, a dense feed-forward of the same
     width in every layer, no side input"""
@@ -143,6 +165,29 @@ def kivorax_fixups(model, cfg):
             model.set_tensor("l%d.mix.left.r2" % i, bits([0.25] * h))
 
 
+def zadinex_fixups(model, cfg):
+    """norms that neither saturate nor drown the token in their offset (else every token would choose the same experts), mixes halfway between the
+    tokens, no correction of the choice, no sink to speak of"""
+    import numpy as np
+
+    def const(name, n, v):
+        model.set_tensor(name, np.full(n, np.float32(v).view(np.uint32) >> 16, dtype=np.uint16))
+    w = cfg["width"]
+    for i, ly in enumerate(cfg["layers"]):
+        for n in ("norm1", "norm2"):
+            const("l%d.%s.b" % (i, n), w, 0.0)
+            const("l%d.%s.alpha" % (i, n), 1, 16.0)
+        if ly["type"] == "wkv":
+            for s in "rkvgw":
+                const("l%d.mix.mu.%s" % (i, s), w, 0.5)
+        else:
+            const("l%d.mix.sink" % i, ly["mixer"]["heads"], -2.0)
+        if ly["mlp"]["kind"] == "moe":
+            const("l%d.mlp.correction" % i, ly["mlp"]["router"]["experts"] + ly["mlp"]["router"]["identity"], 0.0)
+    const("final.norm.b", w, 0.0)
+    const("final.norm.alpha", 1, 16.0)
+
+
 def run(args, ctx, stream):
     import numpy as np
     import torch
@@ -161,7 +206,9 @@ def run(args, ctx, stream):
             ff_active = p["sdt"]["ff"]
             cfgs["sedotar"] = {"hf_config": sedotar_config(p), "gpt": dict(gpt), "init": {"sigma": 0.02, "norm_sigma": 0.02}}
             cfgs["kivorax"] = {"hf_config": kcfg, "gpt": dict(gpt), "init": {"sigma": 0.02, "norm_sigma": 0.02}}
-        if args.compare_arch == "kivorax":
+        if args.compare_arch == "zadinex":
+            cfgs["zadinex"] = {"hf_config": zadinex_config(p), "gpt": dict(gpt), "init": {"sigma": 0.02, "norm_sigma": 0.02}}
+        if args.compare_arch in ("kivorax", "zadinex"):
             kcfg = kivorax_config(p)
             cfgs["kivorax"] = {"hf_config": kcfg, "gpt": {"max_seq_len": P + args.steps + args.warmup + 64, "max_batch": 1, "max_prefill": panel},
                                "init": {"sigma": 0.02, "norm_sigma": 0.02}}
@@ -170,7 +217,7 @@ def run(args, ctx, stream):
         if args.compare_arch == "gadilix":
             cfgs["gadilix"] = {"hf_config": gadilix_config(p), "gpt": dict(gpt), "init": {"sigma": 0.02, "norm_sigma": 0.02}}
             cfgs["sedotar"] = {"hf_config": sedotar_config(p), "gpt": dict(gpt), "init": {"sigma": 0.02, "norm_sigma": 0.02}}
-        if args.compare_arch != "sedotar":
+        if args.compare_arch not in ("sedotar", "zadinex"):
             cfgs["sipazen"] = {"hf_config": sipazen_config(p), "gpt": {"max_seq_len": P + args.steps + args.warmup + 64, "max_batch": 1, "max_prefill": panel},
                                "init": {"sigma": 0.02, "norm_sigma": 0.02}}
         cfgs["qwen3"] = kf.qwen3_config(n_layer, p["width"], (ff_active + 127) // 128 * 128, p["width"] // 128, max(1, p["width"] // 512), 128, p["vocab"], None, False,
@@ -180,6 +227,8 @@ def run(args, ctx, stream):
             model.init_random()
             if name == "kivorax":
                 kivorax_fixups(model, kcfg)
+            if name == "zadinex":
+                zadinex_fixups(model, cfg["hf_config"])
             toks = ((np.arange(P) * 37 + 11) % p["vocab"]).astype(np.int32)
 
             def prompt():
