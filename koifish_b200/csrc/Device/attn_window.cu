@@ -379,22 +379,23 @@ __global__ void __launch_bounds__(AW * 32) kf_attn_window_kernel(WinArgs a) {
 }
 // the splits of one (token, head) merged in split order with the sink, written in the activation type
 __global__ void kf_attn_window_merge_kernel(WinArgs a) {
-    const int m = blockIdx.x, h = blockIdx.y;
+    __shared__ float sf[64];  // nsplit <= 64: factor of every split
+    const int m = blockIdx.x, h = blockIdx.y, lane = threadIdx.x & 31;
     const float* part = a.ws + ((size_t)m * a.H + h) * a.nsplit * (a.dv + 2);
     const float snk = a.sink ? bf16_bits_to_f32(a.sink[h]) : -INFINITY;
-    float Mx = snk;
-    for (int z = 0; z < a.nsplit; z++) Mx = fmaxf(Mx, part[(size_t)z * (a.dv + 2)]);
-    float L = snk == -INFINITY ? 0.f : expf(snk - Mx);
-    for (int z = 0; z < a.nsplit; z++) {
-        const float mz = part[(size_t)z * (a.dv + 2)];
-        if (mz != -INFINITY) L += expf(mz - Mx) * part[(size_t)z * (a.dv + 2) + 1];
-    }
+    // every warp finds the maximum and the denominator on its own; lane z holds splits z and z + 32
+    const int z0 = lane, z1 = lane + 32;
+    const float m0 = z0 < a.nsplit ? part[(size_t)z0 * (a.dv + 2)] : -INFINITY, m1 = z1 < a.nsplit ? part[(size_t)z1 * (a.dv + 2)] : -INFINITY;
+    const float l0 = z0 < a.nsplit ? part[(size_t)z0 * (a.dv + 2) + 1] : 0.f, l1 = z1 < a.nsplit ? part[(size_t)z1 * (a.dv + 2) + 1] : 0.f;
+    const float Mx = fmaxf(snk, warp_max(fmaxf(m0, m1)));
+    const float f0 = m0 == -INFINITY ? 0.f : expf(m0 - Mx), f1 = m1 == -INFINITY ? 0.f : expf(m1 - Mx);
+    const float L = warp_sum(f0 * l0 + f1 * l1) + (snk == -INFINITY ? 0.f : expf(snk - Mx));
+    if (threadIdx.x < 32) sf[z0] = f0, sf[z1] = f1;
+    __syncthreads();
     for (int d = threadIdx.x; d < a.dv; d += blockDim.x) {
         float o = 0.f;
-        for (int z = 0; z < a.nsplit; z++) {
-            const float mz = part[(size_t)z * (a.dv + 2)];
-            if (mz != -INFINITY) o = fmaf(expf(mz - Mx), part[(size_t)z * (a.dv + 2) + 2 + d], o);
-        }
+#pragma unroll 8
+        for (int z = 0; z < a.nsplit; z++) o = fmaf(sf[z], part[(size_t)z * (a.dv + 2) + 2 + d], o);
         win_store(a, m, h, d, o / L);
     }
 }

@@ -40,6 +40,8 @@ struct ScanArgs {
     int unit_qk;             // q, k divided by sqrt(sum x^2 + unit_eps) per head
     int z_head;              // 1: one decay per head and token (z: [H], zbias: [H]) shared by the head's key channels
     float inv_tau, q_scale, unit_eps;
+    int chunk, nch;          // PHASE 1, 2: tokens per chunk, chunks per sequence
+    float *ends, *prods;     // [sequences][nch - 1] x ([H][dv][dk] end states, [H][dk] products of the decays)
 };
 
 // grid (heads, sequences, column chunks).  Thread (pl, r) keeps the NPT (16 or 8) consecutive rows n = r * NPT + i of state column p0 + pl in
@@ -47,8 +49,13 @@ struct ScanArgs {
 // (normalised there), the decay (formed there), v, beta.  FULL (dk == R * NPT): a thread's slice of k, q and the decay is NPT / 4 16-byte
 // shared loads each and nothing is bounds-checked; otherwise rows beyond dk read k = q = 0 and leave their (zero) state alone.
 constexpr int NPT_MAX = 16;
+constexpr int kScanChunk = 64;
 // RULE 0: plain outer-product write; 1: delta-rule write; 2: read-out ahead of the write, with a bonus.
-template <int RULE, bool FULL, int NPT>
+// PHASE 0: a CTA walks all T tokens.  Long panels of the rules whose state map is affine with a diagonal factor (0 and 2) go in two launches over
+// chunks of tokens instead, a CTA per chunk: PHASE 1 leaves every chunk's end state from a zero start and the product of its decays -- chunk
+// 0 starts from the slot's state and is done with its read-outs --, PHASE 2 folds the earlier chunks' maps into a chunk's incoming state,
+// S <- diag(product) S + end, and replays the chunk with read-outs; the last chunk leaves the slot's state, which no CTA of PHASE 2 reads.
+template <int RULE, bool FULL, int NPT, int PHASE>
 __global__ void __launch_bounds__(256) kf_gated_scan_kernel(ScanArgs a) {
     extern __shared__ __align__(16) float sm[];
     constexpr bool DELTA = RULE == 1, BONUS = RULE == 2;
@@ -62,24 +69,40 @@ __global__ void __launch_bounds__(256) kf_gated_scan_kernel(ScanArgs a) {
     float* sV = sG + TB * dkp;       // [TB][PB]
     float* sB = sV + TB * PB;        // [TB]
     float* sKQ = sB + TB;            // [TB] k . q of the staged (normalised, scaled) rows: the delta rule's read-out needs it; RULE 2: (u * k) . q
-    const int h = blockIdx.x, seq = blockIdx.y, p0 = blockIdx.z * PB;
+    const int h = blockIdx.x, seq = PHASE ? blockIdx.y / (a.nch - 1) : blockIdx.y, p0 = blockIdx.z * PB;
+    const int ch = PHASE ? (int)blockIdx.y % (a.nch - 1) + (PHASE == 2 ? 1 : 0) : 0;
+    const int t_lo = PHASE ? ch * a.chunk : 0, t_hi = PHASE ? min(a.T, t_lo + a.chunk) : a.T;
+    const bool emit = PHASE != 1 || ch == 0;
     const int kh = h / (a.H / a.G);
     const int tid = threadIdx.x, pl = tid / R, r = tid - pl * R, p = p0 + pl;
     const bool live = pl < PB && p < a.dv;
     const int m0 = seq * a.T, n0 = r * NPT;
     float* st = a.state + (size_t)a.slot[m0] * a.state_stride + ((size_t)h * a.dv + (live ? p : 0)) * dk;
     const bool fresh = a.pos[m0] == 0;
-    float S[NPT];
+    float S[NPT], P[NPT];
+    if (PHASE == 2) {
+        const size_t es = (size_t)a.H * a.dv * dk, ps = (size_t)a.H * dk;
+        const float* e0 = a.ends + (size_t)seq * (a.nch - 1) * es + ((size_t)h * a.dv + (live ? p : 0)) * dk;
+        const float* q0 = a.prods + (size_t)seq * (a.nch - 1) * ps + (size_t)h * dk;
 #pragma unroll
-    for (int i = 0; i < NPT; i++) S[i] = (live && n0 + i < dk && !fresh) ? st[n0 + i] : 0.f;
+        for (int i = 0; i < NPT; i++) S[i] = (live && n0 + i < dk) ? e0[n0 + i] : 0.f;
+        for (int j = 1; j < ch; j++) {
+#pragma unroll
+            for (int i = 0; i < NPT; i++)
+                if (live && n0 + i < dk) S[i] = fmaf(q0[j * ps + n0 + i], S[i], e0[j * es + n0 + i]);
+        }
+    } else {
+#pragma unroll
+        for (int i = 0; i < NPT; i++) S[i] = (live && n0 + i < dk && !fresh && ch == 0) ? st[n0 + i] : 0.f, P[i] = 1.f;
+    }
     const float Aexp = a.decay_kind == 1 ? expf(bf16_bits_to_f32(a.A_log[h])) : 0.f;
     auto decay = [&](float z) {
         return a.decay_kind == 2 ? expf(-expf(z)) : a.decay_kind == 1 ? expf(-Aexp * softplus_f(z)) : expf(log_sigmoid_f(z) * a.inv_tau);
     };
     const bool zh = a.z_head != 0;  // one decay per head and token: formed once per staged token (sG[tt]), not per key channel
     const int warp = tid >> 5, lane = tid & 31, nwarp = blockDim.x >> 5;
-    for (int t0 = 0; t0 < a.T; t0 += TB) {
-        const int nt = min(TB, a.T - t0);
+    for (int t0 = t_lo; t0 < t_hi; t0 += TB) {
+        const int nt = min(TB, t_hi - t0);
         __syncthreads();
         // four elements per thread and step: their global loads are issued together, then the decays are formed
         for (int i0 = tid; i0 < nt * dk; i0 += 4 * blockDim.x) {
@@ -201,17 +224,26 @@ __global__ void __launch_bounds__(256) kf_gated_scan_kernel(ScanArgs a) {
             for (int i = 0; i < NPT; i++) {
                 if (BONUS) c[i & 3] = fmaf(S[i], qq[i], c[i & 3]);
                 S[i] = fmaf(gg[i], S[i], kk[i] * w);
+                if (PHASE == 1) P[i] *= gg[i];
                 if (!BONUS) c[i & 3] = fmaf(S[i], qq[i], c[i & 3]);
             }
+            if (!emit) continue;
             float acc = (c[0] + c[1]) + (c[2] + c[3]);
             for (int o = R >> 1; o > 0; o >>= 1) acc += __shfl_xor_sync(0xffffffffu, acc, o);
             if (live && r == 0) a.y[(size_t)(m0 + t0 + tt) * a.ldy + h * a.dv + p] = BONUS ? fmaf(sKQ[tt], w, acc) : acc;
         }
     }
-    if (live) {
+    if (!live || (PHASE == 2 && ch != a.nch - 1)) return;
+    float* to = st;
+    if (PHASE == 1) to = a.ends + (((size_t)seq * (a.nch - 1) + ch) * a.H + h) * a.dv * dk + (size_t)p * dk;
+#pragma unroll
+    for (int i = 0; i < NPT; i++)
+        if (n0 + i < dk) to[n0 + i] = S[i];
+    if (PHASE == 1 && p == 0) {
+        float* pr = a.prods + (((size_t)seq * (a.nch - 1) + ch) * a.H + h) * dk;
 #pragma unroll
         for (int i = 0; i < NPT; i++)
-            if (n0 + i < dk) st[n0 + i] = S[i];
+            if (n0 + i < dk) pr[n0 + i] = P[i];
     }
 }
 
@@ -451,14 +483,33 @@ static int scan_launch(kf_ctx* ctx, ScanArgs& a, int nseq, int rule) {
     const size_t smem = (size_t)(3 * TB * dkp + TB * PB + 2 * TB) * sizeof(float);
     KF_REQUIRE(ctx, smem <= 48 * 1024, "staging area");
     a.R = R, a.PB = PB, a.TB = TB, a.dkp = dkp;
-    const dim3 grid(H, nseq, (dv + PB - 1) / PB);
     const bool full = dk == R * NPT;
-#define KF_SCAN(D, F, N) kf_gated_scan_kernel<D, F, N><<<grid, threads, smem, ctx->stream>>>(a)
-#define KF_SCAN_N(D, F) (NPT == 8 ? KF_SCAN(D, F, 8) : KF_SCAN(D, F, 16))
-#define KF_SCAN_R(D) (full ? KF_SCAN_N(D, true) : KF_SCAN_N(D, false))
-    if (rule == 1) KF_SCAN_R(1);
-    else if (rule == 2) KF_SCAN_R(2);
-    else KF_SCAN_R(0);
+    const int cols = (dv + PB - 1) / PB;
+    // long panels: chunks of at least 64 tokens, at most 16 of them
+    const int nch = rule != 1 && T >= 2 * kScanChunk ? std::min(16, T / kScanChunk) : 1;
+    if (nch > 1) {
+        a.chunk = (T + nch - 1) / nch, a.nch = (T + a.chunk - 1) / a.chunk;
+        const size_t ends = (size_t)nseq * (a.nch - 1) * H * dv * dk, prods = (size_t)nseq * (a.nch - 1) * H * dk;
+        KF_REQUIRE(ctx, kf_ensure_attn_ws(ctx, (ends + prods) * sizeof(float)) == KF_OK, "scan workspace");
+        a.ends = ctx->attn_ws, a.prods = a.ends + ends;
+    }
+    const dim3 grid(H, nch > 1 ? nseq * (a.nch - 1) : nseq, cols);
+#define KF_SCAN(D, F, N, P) kf_gated_scan_kernel<D, F, N, P><<<grid, threads, smem, ctx->stream>>>(a)
+#define KF_SCAN_N(D, F, P) (NPT == 8 ? KF_SCAN(D, F, 8, P) : KF_SCAN(D, F, 16, P))
+#define KF_SCAN_R(D, P) (full ? KF_SCAN_N(D, true, P) : KF_SCAN_N(D, false, P))
+    if (nch > 1) {
+        if (rule == 2) KF_SCAN_R(2, 1);
+        else KF_SCAN_R(0, 1);
+        KF_LAUNCH_CHECK(ctx);
+        if (rule == 2) KF_SCAN_R(2, 2);
+        else KF_SCAN_R(0, 2);
+    } else if (rule == 1) {
+        KF_SCAN_R(1, 0);
+    } else if (rule == 2) {
+        KF_SCAN_R(2, 0);
+    } else {
+        KF_SCAN_R(0, 0);
+    }
 #undef KF_SCAN_R
 #undef KF_SCAN_N
 #undef KF_SCAN

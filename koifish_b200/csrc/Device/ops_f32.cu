@@ -116,6 +116,47 @@ __global__ void __launch_bounds__(256) kf_group_norm_kernel(TO* __restrict__ out
     }
 }
 
+// The same for parts of at most 32 * kPartRegs entries that do not go into the residual: a warp per (row, group), its entries in registers.
+constexpr int kPartRegs = 8;
+template <int GATE, typename TO>
+__global__ void __launch_bounds__(256) kf_part_norm_kernel(TO* __restrict__ out, int ldo, const float* __restrict__ x, int ldx, const float* __restrict__ gate, int ldg,
+                                                           const uint16_t* __restrict__ gate_bias, const uint16_t* __restrict__ w, const int32_t* __restrict__ row_idx,
+                                                           int rows, int dim, int groups, float eps, int w_shared, float w_add, float out_mult) {
+    const long long u = (long long)blockIdx.x * 8 + (threadIdx.x >> 5);
+    if (u >= (long long)rows * groups) return;
+    const int r = (int)(u / groups), grp = (int)(u % groups), gs = dim / groups, lane = threadIdx.x & 31;
+    const int src = row_idx ? row_idx[r] : r;
+    const float* xr = x + (size_t)src * ldx + grp * gs;
+    const float* gr = GATE ? gate + (size_t)src * ldg + grp * gs : nullptr;
+    float v[kPartRegs], g[kPartRegs], wt[kPartRegs], ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < kPartRegs; k++) {
+        const int i = lane + 32 * k;
+        const bool in = i < gs;
+        v[k] = in ? xr[i] : 0.f, g[k] = (GATE && in) ? gr[i] : 0.f;
+        wt[k] = in ? bf16_bits_to_f32(w[w_shared == 2 ? 0 : w_shared ? i : grp * gs + i]) : 0.f;
+        if (GATE == 1 && in && gate_bias) g[k] += bf16_bits_to_f32(gate_bias[grp * gs + i]);
+    }
+#pragma unroll
+    for (int k = 0; k < kPartRegs; k++) {
+        if (GATE == 1) v[k] *= sigmoid_f(g[k]);
+        if (GATE == 2) v[k] *= g[k] * sigmoid_f(g[k]);
+        ss = fmaf(v[k], v[k], ss);
+    }
+    const float s = 1.0f / sqrtf(warp_sum(ss) / (float)gs + eps);
+    TO* o = out + (size_t)r * ldo + grp * gs;
+#pragma unroll
+    for (int k = 0; k < kPartRegs; k++) {
+        const int i = lane + 32 * k;
+        if (i >= gs) break;
+        float t = v[k] * s * (w_add + wt[k]);
+        if (GATE == 3) t *= sigmoid_f(g[k]);
+        if (GATE == 4) t *= g[k] * sigmoid_f(g[k]);
+        if (sizeof(TO) == 2) ((uint16_t*)o)[i] = f32_to_bf16_bits(t * out_mult);
+        else ((float*)o)[i] = t * out_mult;
+    }
+}
+
 // Post-norm residual step of one row:  res += mult * v / sqrt(mean(v^2) + eps) * (w_add + w)  with w per entry or (w_one) one number; v is
 //   SRC 0: sa * a + sb * b (b optional);   SRC 1: sum_j wgt[j] * y[entry_slot[j]] + shared (a token's experts; shared optional);
 //   SRC 2: a row of a bf16 table -- then the row starts the stream: res = the normed row.
@@ -383,55 +424,53 @@ __global__ void __launch_bounds__(128) kf_dyt_step_kernel(DytArgs p) {
     const int r = blockIdx.y, i = (blockIdx.x * blockDim.x + threadIdx.x) * V;
     if (i >= p.dim) return;
     const int src = p.row_idx ? p.row_idx[r] : r;
-    float v[V], x[V];
+    float v[V], x[V], s[V], w[V], b[V], d[V], h[V];
+    // everything that does not hang on the experts' places is fetched ahead of them
 #pragma unroll
-    for (int k = 0; k < V; k++) v[k] = 0.f;
+    for (int k = 0; k < V; k++) v[k] = 0.f, s[k] = 1.f;
+    if (SRC != 2 && p.scale) ldb<V>(s, p.scale + i);
+    float al = 0.f;
+    if (p.w) ldb<V>(w, p.w + i), ldb<V>(b, p.b + i), al = bf16_bits_to_f32(*p.alpha);
+    float* tail = p.mu ? p.tail + (size_t)p.slot[r] * p.tail_stride + i : nullptr;
+    const bool first = p.mu && p.pos[r] == 0;
+    if (p.mu) ldf<V>(d, tail);
     if (SRC != 2) ldf<V>(x, p.res + (size_t)src * p.dim + i);
     if (SRC == 0) {
         if (p.a) ldf<V>(v, p.a + (size_t)src * p.lda + i);
     } else if (SRC == 1) {
         const int32_t* es = p.entry_slot + (size_t)src * p.top;
         const float* wg   = p.wgt + (size_t)src * p.top;
-#pragma unroll 4
-        for (int j = 0; j < p.top; j++) {
-            const int sl = es[j];
-            const float wj = wg[j];
-            float t[V];
-            if (sl >= 0) ldf<V>(t, p.y + (size_t)sl * p.dim + i);
-            else ld_actv<TO, V>(t, (const TO*)p.pass + (size_t)src * p.dim + i);
+        float own[V];
+        ld_actv<TO, V>(own, (const TO*)p.pass + (size_t)src * p.dim + i);
+        for (int j0 = 0; j0 < p.top; j0 += 8) {  // eight experts at a time: their places, then their rows, are fetched together
+            int sl[8];
+            float wj[8], t[8][V];
 #pragma unroll
-            for (int k = 0; k < V; k++) v[k] = fmaf(wj, t[k], v[k]);
+            for (int j = 0; j < 8; j++) sl[j] = j0 + j < p.top ? es[j0 + j] : -1, wj[j] = j0 + j < p.top ? wg[j0 + j] : 0.f;
+#pragma unroll
+            for (int j = 0; j < 8; j++)
+                if (sl[j] >= 0) ldf<V>(t[j], p.y + (size_t)sl[j] * p.dim + i);
+#pragma unroll
+            for (int j = 0; j < 8; j++)
+#pragma unroll
+                for (int k = 0; k < V; k++) v[k] = fmaf(wj[j], sl[j] >= 0 ? t[j][k] : own[k], v[k]);
         }
     } else {
         ldb<V>(x, p.table + (size_t)p.tokens[src] * p.dim + i);
     }
     if (SRC != 2) {
-        if (p.scale) {
-            float s[V];
-            ldb<V>(s, p.scale + i);
 #pragma unroll
-            for (int k = 0; k < V; k++) x[k] = fmaf(s[k], v[k], x[k]);
-        } else {
-#pragma unroll
-            for (int k = 0; k < V; k++) x[k] += v[k];
-        }
+        for (int k = 0; k < V; k++) x[k] = fmaf(s[k], v[k], x[k]);
     }
     if (!p.row_idx) stf<V>(p.res + (size_t)r * p.dim + i, x);
     if (!p.w) return;
-    const float al = bf16_bits_to_f32(*p.alpha);
-    float w[V], b[V], h[V];
-    ldb<V>(w, p.w + i), ldb<V>(b, p.b + i);
 #pragma unroll
     for (int k = 0; k < V; k++) h[k] = fmaf(tanhf(al * x[k]), w[k], b[k]);
     if (!p.mu) {
         st_act<TO, V>((TO*)p.out + (size_t)r * p.dim + i, h);
         return;
     }
-    float* tail = p.tail + (size_t)p.slot[r] * p.tail_stride + i;
-    float d[V];
-    ldf<V>(d, tail);
     stf<V>(tail, h);
-    const bool first = p.pos[r] == 0;
 #pragma unroll
     for (int k = 0; k < V; k++) d[k] = (first ? 0.f : d[k]) - h[k];
     for (int q = 0; q < p.n_mix; q++) {
@@ -545,83 +584,133 @@ struct RouteMode {
 };
 constexpr int kRouteGroups = 64;
 // one warp routes one token in kinds 1 and 2.  taken: the token's chosen experts so far (shared or global memory, written by lane 0).
-__device__ __forceinline__ void route_grouped_warp(int* taken, int32_t* idx, float* __restrict__ wgt, const float* __restrict__ lg,
+// Up to 32 * kRouteCache outputs: a lane keeps the scores and choice values of its outputs (lane, lane + 32, ...) in registers and a mask of
+// those taken; more outputs: they are formed again whenever they are looked at.
+constexpr int kRouteCache = 8;
+__device__ __forceinline__ unsigned route_key(float v) {  // unsigned order = float order
+    const unsigned u = __float_as_uint(v);
+    return (u & 0x80000000u) ? ~u : u | 0x80000000u;
+}
+template <bool CACHED>
+__device__ __forceinline__ void route_grouped_body(int* taken, int32_t* idx, float* __restrict__ wgt, const float* __restrict__ lg,
                                                    const uint16_t* __restrict__ bias, int E, int top, const RouteMode md, int lane) {
-    const int per = E / md.groups;
+    const int per = E / md.groups, n = CACHED ? kRouteCache : (E + 31) / 32;
+    float sc[CACHED ? kRouteCache : 1], cv[CACHED ? kRouteCache : 1];
     float mx = 0.f, inv = 1.f;
+    auto shift_of = [&](int e) { return bias ? bf16_bits_to_f32(bias[e]) : 0.f; };
+    if (CACHED) {
+#pragma unroll
+        for (int i = 0; i < kRouteCache; i++) {
+            const int e = lane + 32 * i;
+            sc[i] = e < E ? lg[e] : -INFINITY, cv[i] = e < E ? shift_of(e) : 0.f;
+        }
+    }
     if (md.kind == 2) {
         mx = -INFINITY;
-        for (int e = lane; e < E; e += 32) mx = fmaxf(mx, lg[e]);
-        mx = warp_max(mx);
         float d = 0.f;
-        for (int e = lane; e < E; e += 32) d += expf(lg[e] - mx);
+        if (CACHED) {
+#pragma unroll
+            for (int i = 0; i < kRouteCache; i++) mx = fmaxf(mx, sc[i]);
+            mx = warp_max(mx);
+#pragma unroll
+            for (int i = 0; i < kRouteCache; i++) sc[i] = 32 * i < E ? expf(sc[i] - mx) : 0.f, d += sc[i];
+        } else {
+            for (int e = lane; e < E; e += 32) mx = fmaxf(mx, lg[e]);
+            mx = warp_max(mx);
+            for (int e = lane; e < E; e += 32) d += expf(lg[e] - mx);
+        }
         inv = 1.f / warp_sum(d);
     }
+    if (CACHED) {
+#pragma unroll
+        for (int i = 0; i < kRouteCache; i++)
+            if (32 * i < E) sc[i] = md.kind == 2 ? sc[i] * inv : sigmoid_f(sc[i]), cv[i] += sc[i];
+    }
     auto score  = [&](int e) { return md.kind == 2 ? expf(lg[e] - mx) * inv : sigmoid_f(lg[e]); };
-    auto choice = [&](int e) { return score(e) + (bias ? bf16_bits_to_f32(bias[e]) : 0.f); };
-    unsigned long long kept = 0;
-    if (md.keep >= md.groups) {
-        kept = ~0ull;
-    } else {
-        // lane g & 31 keeps the rank values of groups g and g + 32, found by all lanes together
-        float gs0 = -INFINITY, gs1 = -INFINITY;
+    auto choice = [&](int i, int e) { return CACHED ? cv[CACHED ? i : 0] : score(e) + shift_of(e); };
+    unsigned long long kept = ~0ull;
+    if (md.keep < md.groups) {
+        kept = 0;
+        // lane g & 31 keeps the rank keys of groups g and g + 32, found by all lanes together
+        unsigned gs0 = 0, gs1 = 0;
         for (int g = 0; g < md.groups; g++) {
             float a = -INFINITY, b = -INFINITY;  // largest, second largest of this lane's share
-            for (int e = g * per + lane; e < (g + 1) * per; e += 32) {
-                const float v = choice(e);
+#pragma unroll CACHED ? kRouteCache : 1
+            for (int i = 0; i < n; i++) {
+                const int e = lane + 32 * i;
+                if (e < g * per || e >= (g + 1) * per) continue;
+                const float v = choice(i, e);
                 if (v > a) b = a, a = v;
                 else if (v > b) b = v;
             }
+            float rank;
+            if (md.kind == 1 && per > 1) {
 #pragma unroll
-            for (int o = 16; o > 0; o >>= 1) {
-                const float oa = __shfl_xor_sync(0xffffffffu, a, o), ob = __shfl_xor_sync(0xffffffffu, b, o);
-                const float hi = fmaxf(a, oa), lo = fmaxf(fminf(a, oa), fmaxf(b, ob));
-                a = hi, b = lo;
+                for (int o = 16; o > 0; o >>= 1) {
+                    const float oa = __shfl_xor_sync(0xffffffffu, a, o), ob = __shfl_xor_sync(0xffffffffu, b, o);
+                    const float hi = fmaxf(a, oa), lo = fmaxf(fminf(a, oa), fmaxf(b, ob));
+                    a = hi, b = lo;
+                }
+                rank = a + b;
+            } else {
+                rank = warp_max(a);
             }
-            const float rank = (md.kind == 1 && per > 1) ? a + b : a;
-            if (lane == (g & 31)) (g < 32 ? gs0 : gs1) = rank;
+            if (lane == (g & 31)) (g < 32 ? gs0 : gs1) = route_key(rank);
         }
         for (int r = 0; r < md.keep; r++) {
-            float best = -INFINITY;
-            int bi     = 0x7fffffff;
-            if (lane < md.groups && !((kept >> lane) & 1ull)) best = gs0, bi = lane;
-            if (lane + 32 < md.groups && !((kept >> (lane + 32)) & 1ull) && (bi == 0x7fffffff || gs1 > best)) best = gs1, bi = lane + 32;
-#pragma unroll
-            for (int o = 16; o > 0; o >>= 1) {
-                const float ob = __shfl_xor_sync(0xffffffffu, best, o);
-                const int oi   = __shfl_xor_sync(0xffffffffu, bi, o);
-                if (oi != 0x7fffffff && (bi == 0x7fffffff || ob > best || (ob == best && oi < bi))) best = ob, bi = oi;
-            }
-            if (bi != 0x7fffffff) kept |= 1ull << bi;
+            const bool o0 = lane < md.groups && !((kept >> lane) & 1ull), o1 = lane + 32 < md.groups && !((kept >> (lane + 32)) & 1ull);
+            const unsigned best = __reduce_max_sync(0xffffffffu, max(o0 ? gs0 : 0u, o1 ? gs1 : 0u));
+            const unsigned at = o0 && gs0 == best ? lane : o1 && gs1 == best ? lane + 32 : 0xffffffffu;
+            const unsigned bi = __reduce_min_sync(0xffffffffu, at);  // ties to the lower index
+            if (bi < 64u) kept |= 1ull << bi;
         }
     }
     float sum = 0.f;
-    for (int j = 0; j < top; j++) {
-        float best = -INFINITY;
-        int bi     = 0x7fffffff;
-        for (int e = lane; e < E; e += 32) {
-            if (!((kept >> min(63, e / per)) & 1ull)) continue;
-            bool was = false;
-            for (int q = 0; q < j; q++) was = was || taken[q] == e;
-            if (was) continue;
-            const float v = choice(e);
-            if (bi == 0x7fffffff || v > best || (v == best && e < bi)) best = v, bi = e;
-        }
+    unsigned used = 0;  // CACHED: this lane's outputs that are taken or closed
+    if (CACHED) {
 #pragma unroll
-        for (int o = 16; o > 0; o >>= 1) {
-            const float ob = __shfl_xor_sync(0xffffffffu, best, o);
-            const int oi   = __shfl_xor_sync(0xffffffffu, bi, o);
-            if (oi != 0x7fffffff && (bi == 0x7fffffff || ob > best || (ob == best && oi < bi))) best = ob, bi = oi;
+        for (int i = 0; i < kRouteCache; i++) {
+            const int e = lane + 32 * i;
+            if (e >= E || !((kept >> min(63, e / per)) & 1ull)) used |= 1u << i;
         }
-        if (lane == 0) {
-            const float sc = score(bi);
-            sum += sc;
-            taken[j] = bi, idx[j] = bi, wgt[j] = md.kind == 2 ? sc : md.scale * sc;
+    }
+    for (int j = 0; j < top; j++) {
+        unsigned bk = 0, bi = 0xffffffffu;
+        float bs = 0.f;
+#pragma unroll CACHED ? kRouteCache : 1
+        for (int i = 0; i < n; i++) {
+            const int e = lane + 32 * i;
+            if (CACHED) {
+                if ((used >> i) & 1u) continue;
+            } else {
+                if (e >= E || !((kept >> min(63, e / per)) & 1ull)) continue;
+                bool was = false;
+                for (int q = 0; q < j; q++) was = was || taken[q] == e;
+                if (was) continue;
+            }
+            const unsigned k = route_key(choice(i, e));
+            if (bi == 0xffffffffu || k > bk) bk = k, bi = e, bs = CACHED ? sc[CACHED ? i : 0] : 0.f;
         }
+        const unsigned best = __reduce_max_sync(0xffffffffu, bk);
+        const unsigned win  = __reduce_min_sync(0xffffffffu, bk == best ? bi : 0xffffffffu);
+        const int w = (int)min(win, (unsigned)(E - 1));
+        if (CACHED) {
+            bs = __shfl_sync(0xffffffffu, bs, w & 31);
+            if (lane == (w & 31)) used |= 1u << (w >> 5);
+        } else {
+            bs = score(w);
+        }
+        sum += bs;
+        if (lane == 0) taken[j] = w, idx[j] = w, wgt[j] = md.kind == 2 ? bs : md.scale * bs;
         __syncwarp();
     }
     if (md.kind == 2 && lane == 0)
         for (int j = 0; j < top; j++) wgt[j] /= sum + 1e-20f;
+}
+__device__ __forceinline__ void route_grouped_warp(int* taken, int32_t* idx, float* __restrict__ wgt, const float* __restrict__ lg,
+                                                   const uint16_t* __restrict__ bias, int E, int top, const RouteMode md, int lane) {
+    if (E <= 32 * kRouteCache) route_grouped_body<true>(taken, idx, wgt, lg, bias, E, top, md, lane);
+    else route_grouped_body<false>(taken, idx, wgt, lg, bias, E, top, md, lane);
 }
 // one warp per token: `top` rounds of arg-max over the E router logits (+ bias), ties to the lower index; weights = softmax over the
 // chosen logits only, or (full) the chosen entries of the softmax over ALL experts, not renormalised.  All in fp32.
@@ -685,7 +774,7 @@ __device__ __forceinline__ void dispatch_small(const int* sidx, int* srank, int 
         for (int e0 = 0; e0 < E; e0 += 32) {
             const int e = e0 + lane;
             int c = 0;
-            for (int j = 0; j < n; j++) c += sidx[j] == e;  // e >= E matches nothing
+            for (int j = 0; j < n; j++) c += sidx[j] == e && e < E;  // outputs beyond the experts take no slot
             int incl = c;
 #pragma unroll
             for (int o = 1; o < 32; o <<= 1) {
@@ -937,7 +1026,15 @@ extern "C" int kf_group_rmsnorm_wadd(kf_ctx* ctx, void* out, int out_kind, int l
     dim3 grid(rows, groups);
     const uint16_t *gb = (const uint16_t*)gate_bias_bf16, *w = (const uint16_t*)w_bf16;
 #define KF_GN(G, A, T) kf_group_norm_kernel<G, A, T><<<grid, 256, 0, ctx->stream>>>((T*)out, ldo, res, x, ldx, gate, ldg, gb, w, row_idx, dim, groups, eps, mult, w_shared, w_add, out_mult)
-    if (out_kind == 2) {
+    if (out_kind != 2 && groups > 1 && dim / groups <= 32 * kPartRegs) {
+        const unsigned blocks = (unsigned)(((long long)rows * groups + 7) / 8);
+#define KF_PART(G, T) kf_part_norm_kernel<G, T><<<blocks, 256, 0, ctx->stream>>>((T*)out, ldo, x, ldx, gate, ldg, gb, w, row_idx, rows, dim, groups, eps, w_shared, w_add, out_mult)
+#define KF_PART_G(T) (gate_kind == 0 ? KF_PART(0, T) : gate_kind == 1 ? KF_PART(1, T) : gate_kind == 2 ? KF_PART(2, T) : gate_kind == 3 ? KF_PART(3, T) : KF_PART(4, T))
+        if (out_kind == 1) KF_PART_G(float);
+        else KF_PART_G(uint16_t);
+#undef KF_PART_G
+#undef KF_PART
+    } else if (out_kind == 2) {
         if (gate_kind == 0) KF_GN(0, true, float);
         else if (gate_kind == 1) KF_GN(1, true, float);
         else if (gate_kind == 2) KF_GN(2, true, float);
