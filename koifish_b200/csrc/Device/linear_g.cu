@@ -157,6 +157,66 @@ __global__ void __launch_bounds__(256) kf_lin_gemv_batch_kernel(BatchArgs a) {
     if (lane == 0) a.y[j][(size_t)row * a.ldy[j] + n] = lin_act(s, a.act[j]);
 }
 
+// Few outputs over a long reduction for a panel of rows (a router, a low-rank projection): a warp takes kSkC outputs of kSkR rows, so a weight
+// fragment serves kSkR rows and a row fragment kSkC outputs.  Row lengths are multiples of 8 and everything is 16-byte aligned.
+constexpr int kSkR = 4, kSkC = 2;
+template <typename TA>
+__global__ void __launch_bounds__(256) kf_lin_skinny_kernel(LinArgs a) {
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int n0 = (blockIdx.x * 8 + warp) * kSkC, m0 = blockIdx.y * kSkR;
+    if (n0 >= a.N) return;
+    const uint16_t* w[kSkC];
+    const TA* x[kSkR];
+#pragma unroll
+    for (int j = 0; j < kSkC; j++) w[j] = a.W0 + (size_t)min(n0 + j, a.N - 1) * a.K;
+#pragma unroll
+    for (int i = 0; i < kSkR; i++) x[i] = (const TA*)a.x + (size_t)min(m0 + i, a.M - 1) * a.ldx;
+    float s[kSkR][kSkC];
+#pragma unroll
+    for (int i = 0; i < kSkR; i++)
+#pragma unroll
+        for (int j = 0; j < kSkC; j++) s[i][j] = 0.f;
+#pragma unroll 2
+    for (int k = lane * 8; k < a.K; k += 256) {
+        float wv[kSkC][8];
+#pragma unroll
+        for (int j = 0; j < kSkC; j++) {
+            const uint4 q = *reinterpret_cast<const uint4*>(w[j] + k);
+            const uint32_t u[4] = {q.x, q.y, q.z, q.w};
+#pragma unroll
+            for (int e = 0; e < 4; e++) wv[j][2 * e] = bf16lo(u[e]), wv[j][2 * e + 1] = bf16hi(u[e]);
+        }
+#pragma unroll
+        for (int i = 0; i < kSkR; i++) {
+            float xv[8];
+            if (sizeof(TA) == 2) {
+                const uint4 q = *reinterpret_cast<const uint4*>((const uint16_t*)x[i] + k);
+                const uint32_t u[4] = {q.x, q.y, q.z, q.w};
+#pragma unroll
+                for (int e = 0; e < 4; e++) xv[2 * e] = bf16lo(u[e]), xv[2 * e + 1] = bf16hi(u[e]);
+            } else {
+                const float4 f0 = *reinterpret_cast<const float4*>((const float*)x[i] + k), f1 = *reinterpret_cast<const float4*>((const float*)x[i] + k + 4);
+                xv[0] = f0.x, xv[1] = f0.y, xv[2] = f0.z, xv[3] = f0.w, xv[4] = f1.x, xv[5] = f1.y, xv[6] = f1.z, xv[7] = f1.w;
+            }
+#pragma unroll
+            for (int j = 0; j < kSkC; j++)
+#pragma unroll
+                for (int e = 0; e < 8; e++) s[i][j] = fmaf(wv[j][e], xv[e], s[i][j]);
+        }
+    }
+#pragma unroll
+    for (int i = 0; i < kSkR; i++)
+#pragma unroll
+        for (int j = 0; j < kSkC; j++) {
+            const float t = warp_sum(s[i][j]);
+            if (lane == 0 && m0 + i < a.M && n0 + j < a.N) {
+                const float r = lin_act(t, a.act);
+                if (a.act && a.out_act == 1) ((uint16_t*)a.y)[(size_t)(m0 + i) * a.ldy + n0 + j] = f32_to_bf16_bits(r);
+                else ((float*)a.y)[(size_t)(m0 + i) * a.ldy + n0 + j] = r;
+            }
+        }
+}
+
 // ------------------------------------------------------------------------------------------------------------------ tile kernel
 // 64 slots x 64 outputs per CTA, k in steps of 64 (bf16) or 32 (float); 256 threads.  Float activations: each thread a 4 x 4 block of FFMA accumulators.
 // bf16 activations: 8 warps as 4 (m) x 2 (n), each warp 16 x 32 through mma.sync.m16n8k16; operands come from the same shared tiles.
@@ -347,21 +407,31 @@ int dispatch(kf_ctx* ctx, const LinArgs& a, int slots, int groups, bool gemv, bo
     return dual ? launch<uint16_t, true>(ctx, a, slots, groups, gemv) : launch<uint16_t, false>(ctx, a, slots, groups, gemv);
 }
 constexpr int kGemvMaxSlots = 16;
+// one weight, a panel of rows, few outputs and a long reduction: tiles would leave all but a handful of SMs idle
+bool skinny_shape(const LinArgs& a) { return a.N <= 128 && a.K >= 512 && a.M > kGemvMaxSlots; }
+int dispatch_one(kf_ctx* ctx, const LinArgs& a, int act_f32) {
+    const bool skinny = skinny_shape(a);
+    if (skinny && a.K % 8 == 0 && a.ldx % 8 == 0 && (((uintptr_t)a.W0 | (uintptr_t)a.x) & 15) == 0 && (a.M + kSkR - 1) / kSkR <= 65535) {
+        const dim3 grid((a.N + 8 * kSkC - 1) / (8 * kSkC), (a.M + kSkR - 1) / kSkR);
+        if (act_f32) kf_lin_skinny_kernel<float><<<grid, 256, 0, ctx->stream>>>(a);
+        else kf_lin_skinny_kernel<uint16_t><<<grid, 256, 0, ctx->stream>>>(a);
+        KF_LAUNCH_CHECK(ctx);
+        return KF_OK;
+    }
+    return dispatch(ctx, a, a.M, 1, a.M <= kGemvMaxSlots || (skinny && a.N <= 64), false, act_f32);
+}
 }  // namespace
 
 extern "C" int kf_linear_g(kf_ctx* ctx, float* y, int ldy, const kf_tensor_desc* w, const void* x, int act_f32, int ldx, int M) {
     if (!ctx || !y || !w || !x) return KF_ERR_BAD_ARG;
     KF_REQUIRE(ctx, w->type == KF_T_BF16 && M >= 1 && w->rows >= 1 && w->cols >= 1 && ldx >= w->cols && ldy >= w->rows, "bf16 weight, ld >= extent");
-    // few outputs over a long reduction (a gate or a router of a panel): tiles would leave all but a handful of SMs idle, so every
-    // (token, output) pair gets a warp instead; the weight (<= 64 rows) stays in L2
-    const bool skinny = w->rows <= 64 && w->cols >= 512 && M > kGemvMaxSlots;
-    // shapes the tuned kernels take go there (tcgen05 / TMEM panels, the HBM-rate GEMV); fp32 result through their fp32 epilogue
-    if (!skinny && !act_f32 && ldx == w->cols && ldy == w->rows && w->cols % 128 == 0 && w->rows % 16 == 0 && w->rows >= 16 && ctx->tc_min_m != 0 &&
-        (((uintptr_t)w->data_dev | (uintptr_t)x | (uintptr_t)y) & 15) == 0)
-        return kf_linear(ctx, y, w, x, M, KF_EPI_F32, nullptr);
     LinArgs a = {};
     a.W0 = (const uint16_t*)w->data_dev, a.x = x, a.y = y, a.M = M, a.N = w->rows, a.K = w->cols, a.ldx = ldx, a.ldy = ldy;
-    return dispatch(ctx, a, M, 1, M <= kGemvMaxSlots || skinny, false, act_f32);
+    // shapes the tuned kernels take go there (tcgen05 / TMEM panels, the HBM-rate GEMV); fp32 result through their fp32 epilogue
+    if (!skinny_shape(a) && !act_f32 && ldx == w->cols && ldy == w->rows && w->cols % 128 == 0 && w->rows % 16 == 0 && w->rows >= 16 && ctx->tc_min_m != 0 &&
+        (((uintptr_t)w->data_dev | (uintptr_t)x | (uintptr_t)y) & 15) == 0)
+        return kf_linear(ctx, y, w, x, M, KF_EPI_F32, nullptr);
+    return dispatch_one(ctx, a, act_f32);
 }
 // y = silu(Wg x) * (Wu x), written in the activation type (bf16 bits, or float when act_f32)
 extern "C" int kf_linear_g_swiglu(kf_ctx* ctx, void* y, int ldy, const kf_tensor_desc* wg, const kf_tensor_desc* wu, const void* x, int act_f32,
@@ -427,7 +497,7 @@ extern "C" int kf_linear_batch(kf_ctx* ctx, int n, float* const* y, const kf_ten
             if (act && act[i]) {
                 LinArgs a = {};
                 a.W0 = (const uint16_t*)w[i].data_dev, a.x = x[i], a.y = y[i], a.M = M, a.N = w[i].rows, a.K = w[i].cols, a.ldx = ldx, a.ldy = w[i].rows, a.act = act[i];
-                rc = dispatch(ctx, a, M, 1, w[i].rows <= 64 && w[i].cols >= 512, false, act_f32);
+                rc = dispatch_one(ctx, a, act_f32);
             } else {
                 rc = kf_linear_g(ctx, y[i], w[i].rows, &w[i], x[i], act_f32, ldx, M);
             }

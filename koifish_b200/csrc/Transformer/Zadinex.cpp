@@ -261,8 +261,7 @@ static int BuildZadinex(Fish& f) {
             }
             KF_TRY(b.Buf(&e->tables, (size_t)3 * mc.experts * sizeof(void*)));
             maxE = std::max<size_t>(maxE, mc.experts + mc.pass), maxTop = std::max<size_t>(maxTop, mc.top), maxH1 = std::max<size_t>(maxH1, (size_t)mc.top * mc.ff);
-            KF_TRY(b.Stack(blk->router, {e->router}));
-            maxU = std::max<size_t>(maxU, blk->router.rows);
+            maxU = std::max<size_t>(maxU, mc.experts + mc.pass);
             blk->moe = std::move(e);
         }
         f.blocks.push_back(std::move(blk));
@@ -310,7 +309,6 @@ static int PrepareZadinex(Fish& f) {
         ZdxBlock* b = BlockOf(f, i);
         int rc = b->wkv ? b->wkv->mus.Fill(f.ctx) : b->cat.Fill(f.ctx);
         if (!rc && b->dense) rc = b->dense->cat.Fill(f.ctx);
-        if (!rc && b->moe) rc = b->router.Fill(f.ctx);
         if (!rc && b->moe) rc = b->moe->Prepare();
         if (rc) return rc;
     }
@@ -444,8 +442,9 @@ static int ForwardZadinex(Fish& f, int M, bool want_logits) {
         if (blk->dense) {
             KF_TRY(blk->dense->cuInfer(M));
         } else {
-            KF_TRY(LinStacked(f, s.u, blk->router, s.hact, M));
-            KF_TRY(blk->moe->Route(M, s.u, blk->router.rows, 0));
+            const int outs = blk->moe->card.experts + blk->moe->card.pass;
+            KF_TRY(Lin(f, s.u, outs, blk->moe->router, s.hact, E, M));
+            KF_TRY(blk->moe->Route(M, s.u, outs, 0));
             KF_TRY(blk->moe->Experts(M, s.offsets, s.slot_row, s.slot_group));
             added_moe = blk->moe.get();  // combined by the step that adds it
         }

@@ -49,8 +49,7 @@ struct GeluFF : GeNeuron {  // W_down (gelu(W_gate h) * (W_up h)), gelu in its t
 struct ZdxBlock : GeNeuron {
     TanhNorm norm1, norm2;
     hGTensor ls1, ls2;
-    StackedLinear cat;     // attention: q | k | v
-    StackedLinear router;  // alone, padded to the row count that the tuned matmuls take
+    StackedLinear cat;  // attention: q | k | v
     std::unique_ptr<TimeMix> wkv;
     std::unique_ptr<BlendedAttention> attn;
     std::unique_ptr<GeluFF> dense;
