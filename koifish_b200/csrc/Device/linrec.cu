@@ -40,6 +40,7 @@ struct ScanArgs {
     int unit_qk;             // q, k divided by sqrt(sum x^2 + unit_eps) per head
     int z_head;              // 1: one decay per head and token (z: [H], zbias: [H]) shared by the head's key channels
     float inv_tau, q_scale, unit_eps;
+    int vec;                 // 1: rows, row lengths and strides allow 16-byte loads
     int chunk, nch;          // PHASE 1, 2: tokens per chunk, chunks per sequence
     float *ends, *prods;     // [sequences][nch - 1] x ([H][dv][dk] end states, [H][dk] products of the decays)
 };
@@ -50,19 +51,19 @@ struct ScanArgs {
 // shared loads each and nothing is bounds-checked; otherwise rows beyond dk read k = q = 0 and leave their (zero) state alone.
 constexpr int NPT_MAX = 16;
 constexpr int kScanChunk = 64;
+constexpr int kScanStep = 4;  // rules 0 and 2: read-outs of this many tokens are reduced over the lanes together
 // RULE 0: plain outer-product write; 1: delta-rule write; 2: read-out ahead of the write, with a bonus.
 // PHASE 0: a CTA walks all T tokens.  Long panels of the rules whose state map is affine with a diagonal factor (0 and 2) go in two launches over
 // chunks of tokens instead, a CTA per chunk: PHASE 1 leaves every chunk's end state from a zero start and the product of its decays -- chunk
 // 0 starts from the slot's state and is done with its read-outs --, PHASE 2 folds the earlier chunks' maps into a chunk's incoming state,
 // S <- diag(product) S + end, and replays the chunk with read-outs; the last chunk leaves the slot's state, which no CTA of PHASE 2 reads.
 template <int RULE, bool FULL, int NPT, int PHASE>
-__global__ void __launch_bounds__(256) kf_gated_scan_kernel(ScanArgs a) {
+__global__ void __launch_bounds__(256, NPT == 8 ? 3 : 2) kf_gated_scan_kernel(ScanArgs a) {
     extern __shared__ __align__(16) float sm[];
     constexpr bool DELTA = RULE == 1, BONUS = RULE == 2;
-    // staged rows are padded by 4 floats after every 16: the R lanes of a column read slices 20 floats apart, which fall into different
-    // banks (slices exactly 16 apart would collide two by two)
+    // staged rows are padded by 4 floats after every 32: the slices (8 or 16 floats apart) of up to 8 neighbouring lanes fall into different banks
     const int dk = a.dk, TB = a.TB, PB = a.PB, R = a.R, dkp = a.dkp;
-    auto ix = [](int n) { return n + ((n >> 4) << 2); };
+    auto ix = [](int n) { return n + ((n >> 5) << 2); };
     float* sK = sm;                  // [TB][dkp]
     float* sQ = sK + TB * dkp;       // [TB][dkp]
     float* sG = sQ + TB * dkp;       // [TB][dkp]
@@ -79,7 +80,7 @@ __global__ void __launch_bounds__(256) kf_gated_scan_kernel(ScanArgs a) {
     const int m0 = seq * a.T, n0 = r * NPT;
     float* st = a.state + (size_t)a.slot[m0] * a.state_stride + ((size_t)h * a.dv + (live ? p : 0)) * dk;
     const bool fresh = a.pos[m0] == 0;
-    float S[NPT], P[NPT];
+    float S[NPT], P[PHASE == 1 ? NPT : 1];
     if (PHASE == 2) {
         const size_t es = (size_t)a.H * a.dv * dk, ps = (size_t)a.H * dk;
         const float* e0 = a.ends + (size_t)seq * (a.nch - 1) * es + ((size_t)h * a.dv + (live ? p : 0)) * dk;
@@ -93,8 +94,11 @@ __global__ void __launch_bounds__(256) kf_gated_scan_kernel(ScanArgs a) {
         }
     } else {
 #pragma unroll
-        for (int i = 0; i < NPT; i++) S[i] = (live && n0 + i < dk && !fresh && ch == 0) ? st[n0 + i] : 0.f, P[i] = 1.f;
+        for (int i = 0; i < NPT; i++) S[i] = (live && n0 + i < dk && !fresh && ch == 0) ? st[n0 + i] : 0.f;
     }
+    if (PHASE == 1)
+#pragma unroll
+        for (int i = 0; i < NPT; i++) P[PHASE == 1 ? i : 0] = 1.f;
     const float Aexp = a.decay_kind == 1 ? expf(bf16_bits_to_f32(a.A_log[h])) : 0.f;
     auto decay = [&](float z) {
         return a.decay_kind == 2 ? expf(-expf(z)) : a.decay_kind == 1 ? expf(-Aexp * softplus_f(z)) : expf(log_sigmoid_f(z) * a.inv_tau);
@@ -104,26 +108,60 @@ __global__ void __launch_bounds__(256) kf_gated_scan_kernel(ScanArgs a) {
     for (int t0 = t_lo; t0 < t_hi; t0 += TB) {
         const int nt = min(TB, t_hi - t0);
         __syncthreads();
-        // four elements per thread and step: their global loads are issued together, then the decays are formed
-        for (int i0 = tid; i0 < nt * dk; i0 += 4 * blockDim.x) {
-            float kv[4], qv[4], zv[4];
+        if (a.vec) {  // four neighbouring entries per access
+            const int d4 = dk >> 2, n4 = nt * d4;
+            for (int i0 = tid; i0 < n4; i0 += 2 * blockDim.x) {
+                float4 kv[2], qv[2], zv[2];
+                int at[2];
 #pragma unroll
-            for (int e = 0; e < 4; e++) {
-                const int i = i0 + e * blockDim.x;
-                if (i < nt * dk) {
-                    const int tt = i / dk, n = i - tt * dk;
-                    const size_t m = (size_t)(m0 + t0 + tt);
-                    kv[e] = a.k[m * a.ldk + kh * dk + n], qv[e] = a.q[m * a.ldq + kh * dk + n];
-                    if (!zh) zv[e] = a.z[m * a.ldz + h * dk + n] + (a.zbias ? bf16_bits_to_f32(a.zbias[h * dk + n]) : 0.f);
+                for (int e = 0; e < 2; e++) {
+                    const int i = i0 + e * blockDim.x;
+                    if (i < n4) {
+                        const int tt = i / d4, n = (i - tt * d4) * 4;
+                        const size_t m = (size_t)(m0 + t0 + tt);
+                        at[e] = tt * dkp + ix(n);
+                        kv[e] = *reinterpret_cast<const float4*>(a.k + m * a.ldk + kh * dk + n);
+                        if (emit) qv[e] = *reinterpret_cast<const float4*>(a.q + m * a.ldq + kh * dk + n);
+                        if (!zh) {
+                            zv[e] = *reinterpret_cast<const float4*>(a.z + m * a.ldz + h * dk + n);
+                            if (a.zbias) {
+                                const uint2 b = *reinterpret_cast<const uint2*>(a.zbias + h * dk + n);
+                                zv[e].x += bf16lo(b.x), zv[e].y += bf16hi(b.x), zv[e].z += bf16lo(b.y), zv[e].w += bf16hi(b.y);
+                            }
+                        }
+                    }
+                }
+#pragma unroll
+                for (int e = 0; e < 2; e++) {
+                    if (i0 + e * blockDim.x < n4) {
+                        *reinterpret_cast<float4*>(sK + at[e]) = kv[e];
+                        if (emit) *reinterpret_cast<float4*>(sQ + at[e]) = qv[e];
+                        if (!zh) *reinterpret_cast<float4*>(sG + at[e]) = make_float4(decay(zv[e].x), decay(zv[e].y), decay(zv[e].z), decay(zv[e].w));
+                    }
                 }
             }
+        } else {
+            // four elements per thread and step: their global loads are issued together, then the decays are formed
+            for (int i0 = tid; i0 < nt * dk; i0 += 4 * blockDim.x) {
+                float kv[4], qv[4], zv[4];
 #pragma unroll
-            for (int e = 0; e < 4; e++) {
-                const int i = i0 + e * blockDim.x;
-                if (i < nt * dk) {
-                    const int tt = i / dk, o = tt * dkp + ix(i - tt * dk);
-                    sK[o] = kv[e], sQ[o] = qv[e];
-                    if (!zh) sG[o] = decay(zv[e]);
+                for (int e = 0; e < 4; e++) {
+                    const int i = i0 + e * blockDim.x;
+                    if (i < nt * dk) {
+                        const int tt = i / dk, n = i - tt * dk;
+                        const size_t m = (size_t)(m0 + t0 + tt);
+                        kv[e] = a.k[m * a.ldk + kh * dk + n], qv[e] = a.q[m * a.ldq + kh * dk + n];
+                        if (!zh) zv[e] = a.z[m * a.ldz + h * dk + n] + (a.zbias ? bf16_bits_to_f32(a.zbias[h * dk + n]) : 0.f);
+                    }
+                }
+#pragma unroll
+                for (int e = 0; e < 4; e++) {
+                    const int i = i0 + e * blockDim.x;
+                    if (i < nt * dk) {
+                        const int tt = i / dk, o = tt * dkp + ix(i - tt * dk);
+                        sK[o] = kv[e], sQ[o] = qv[e];
+                        if (!zh) sG[o] = decay(zv[e]);
+                    }
                 }
             }
         }
@@ -146,62 +184,60 @@ __global__ void __launch_bounds__(256) kf_gated_scan_kernel(ScanArgs a) {
         if (DELTA)
             for (int i = tid; i < nt; i += blockDim.x) sB[i] = sigmoid_f(a.beta[(size_t)(m0 + t0 + i) * a.ldb + h]);
         __syncthreads();
-        // unit vectors / query scale: one warp per staged token
-        for (int tt = warp; tt < nt; tt += nwarp) {
-            float sq = 0.f, sk = 0.f;
-            if (a.unit_qk) {
-                for (int n = lane; n < dk; n += 32) sq = fmaf(sQ[tt * dkp + ix(n)], sQ[tt * dkp + ix(n)], sq), sk = fmaf(sK[tt * dkp + ix(n)], sK[tt * dkp + ix(n)], sk);
-                sq = warp_sum(sq), sk = warp_sum(sk);
+        // unit vectors / query scale: one warp per staged token (nothing to do for plain rows with factor 1)
+        if (DELTA || a.unit_qk || ((BONUS || a.q_scale != 1.f) && emit)) {
+            for (int tt = warp; tt < nt; tt += nwarp) {
+                float sq = 0.f, sk = 0.f;
+                if (a.unit_qk) {
+                    for (int n = lane; n < dk; n += 32) sq = fmaf(sQ[tt * dkp + ix(n)], sQ[tt * dkp + ix(n)], sq), sk = fmaf(sK[tt * dkp + ix(n)], sK[tt * dkp + ix(n)], sk);
+                    sq = warp_sum(sq), sk = warp_sum(sk);
+                }
+                const float fq = a.unit_qk ? a.q_scale / sqrtf(sq + a.unit_eps) : a.q_scale;
+                const float fk = a.unit_qk ? 1.f / sqrtf(sk + a.unit_eps) : 1.f;
+                float kq = 0.f;
+                for (int n = lane; n < dk; n += 32) {
+                    const float qn = sQ[tt * dkp + ix(n)] * fq, kn = sK[tt * dkp + ix(n)] * fk;
+                    if (!BONUS) sQ[tt * dkp + ix(n)] = qn;
+                    if (a.unit_qk) sK[tt * dkp + ix(n)] = kn;
+                    kq = fmaf(BONUS ? bf16_bits_to_f32(a.bonus[h * dk + n]) * kn : kn, qn, kq);
+                }
+                if (DELTA || BONUS) {
+                    kq = warp_sum(kq);
+                    if (lane == 0) sKQ[tt] = kq;
+                }
             }
-            const float fq = a.unit_qk ? a.q_scale / sqrtf(sq + a.unit_eps) : a.q_scale;
-            const float fk = a.unit_qk ? 1.f / sqrtf(sk + a.unit_eps) : 1.f;
-            float kq = 0.f;
-            for (int n = lane; n < dk; n += 32) {
-                const float qn = sQ[tt * dkp + ix(n)] * fq, kn = sK[tt * dkp + ix(n)] * fk;
-                sQ[tt * dkp + ix(n)] = qn;
-                if (a.unit_qk) sK[tt * dkp + ix(n)] = kn;
-                kq = fmaf(BONUS ? bf16_bits_to_f32(a.bonus[h * dk + n]) * kn : kn, qn, kq);
-            }
-            if (DELTA || BONUS) {
-                kq = warp_sum(kq);
-                if (lane == 0) sKQ[tt] = kq;
-            }
+            __syncthreads();
         }
-        __syncthreads();
-        for (int tt = 0; tt < nt; tt++) {
-            float kk[NPT], qq[NPT], gg[NPT];
+        // this thread's slice of a staged row
+        auto slice = [&](float (&to)[NPT], const float* rows, int tt, float beyond) {
             if (FULL) {
-                const float4* k4 = reinterpret_cast<const float4*>(sK + tt * dkp + ix(n0));
-                const float4* q4 = reinterpret_cast<const float4*>(sQ + tt * dkp + ix(n0));
-                const float4* g4 = reinterpret_cast<const float4*>(sG + tt * dkp + ix(n0));
+                // a slice of 16 that starts at a multiple of 16 never crosses the padding
+                const float4* f4 = reinterpret_cast<const float4*>(rows + tt * dkp + ix(n0));
 #pragma unroll
                 for (int j = 0; j < NPT / 4; j++) {
-                    const float4 kv = k4[j], qv = q4[j];
-                    kk[4 * j] = kv.x, kk[4 * j + 1] = kv.y, kk[4 * j + 2] = kv.z, kk[4 * j + 3] = kv.w;
-                    qq[4 * j] = qv.x, qq[4 * j + 1] = qv.y, qq[4 * j + 2] = qv.z, qq[4 * j + 3] = qv.w;
-                }
-                if (zh) {
-                    const float gh = sG[tt];
-#pragma unroll
-                    for (int i = 0; i < NPT; i++) gg[i] = gh;
-                } else {
-#pragma unroll
-                    for (int j = 0; j < NPT / 4; j++) {
-                        const float4 gv = g4[j];
-                        gg[4 * j] = gv.x, gg[4 * j + 1] = gv.y, gg[4 * j + 2] = gv.z, gg[4 * j + 3] = gv.w;
-                    }
+                    const float4 f = f4[j];
+                    to[4 * j] = f.x, to[4 * j + 1] = f.y, to[4 * j + 2] = f.z, to[4 * j + 3] = f.w;
                 }
             } else {
 #pragma unroll
-                for (int i = 0; i < NPT; i++) {
-                    const bool in = n0 + i < dk;
-                    const int o = tt * dkp + ix(n0 + i);
-                    kk[i] = in ? sK[o] : 0.f, qq[i] = in ? sQ[o] : 0.f, gg[i] = in ? sG[zh ? tt : o] : 1.f;
-                }
+                for (int i = 0; i < NPT; i++) to[i] = n0 + i < dk ? rows[tt * dkp + ix(n0 + i)] : beyond;
             }
-            const float vv = sV[tt * PB + (pl < PB ? pl : 0)];
-            float w = vv;
-            if (DELTA) {
+        };
+        auto decays = [&](float (&gg)[NPT], int tt) {
+            if (!zh) {
+                slice(gg, sG, tt, 1.f);
+            } else {
+                const float gh = sG[tt];
+#pragma unroll
+                for (int i = 0; i < NPT; i++) gg[i] = gh;
+            }
+        };
+        float* yt = a.y + (size_t)(m0 + t0) * a.ldy + h * a.dv + p;
+        const int pv = pl < PB ? pl : 0;
+        if (DELTA) {
+            for (int tt = 0; tt < nt; tt++) {
+                float kk[NPT], qq[NPT], gg[NPT];
+                slice(kk, sK, tt, 0.f), slice(qq, sQ, tt, 0.f), decays(gg, tt);
                 // With D = diag(g) S the write is S' = D + k w^T, so the read-out S'^T q = D^T q + (k . q) w: both sums run over D in ONE pass
                 // (two independent chains, their cross-lane sums interleaved) instead of a second pass over S' that waits for w.
                 float d[4] = {0.f, 0.f, 0.f, 0.f}, e[4] = {0.f, 0.f, 0.f, 0.f};  // four partial sums each: the chains are 4 deep, not 16
@@ -213,24 +249,49 @@ __global__ void __launch_bounds__(256) kf_gated_scan_kernel(ScanArgs a) {
                 }
                 float dot = (d[0] + d[1]) + (d[2] + d[3]), rd = (e[0] + e[1]) + (e[2] + e[3]);
                 for (int o = R >> 1; o > 0; o >>= 1) dot += __shfl_xor_sync(0xffffffffu, dot, o), rd += __shfl_xor_sync(0xffffffffu, rd, o);
-                w = sB[tt] * (vv - dot);
+                const float w = sB[tt] * (sV[tt * PB + pv] - dot);
 #pragma unroll
                 for (int i = 0; i < NPT; i++) S[i] = fmaf(kk[i], w, S[i]);
-                if (live && r == 0) a.y[(size_t)(m0 + t0 + tt) * a.ldy + h * a.dv + p] = fmaf(sKQ[tt], w, rd);
-                continue;
+                if (live && r == 0) yt[(size_t)tt * a.ldy] = fmaf(sKQ[tt], w, rd);
             }
-            float c[4] = {0.f, 0.f, 0.f, 0.f};
+            continue;
+        }
+        for (int tt = 0; tt < nt; tt += kScanStep) {
+            float acc[kScanStep], w[kScanStep];
 #pragma unroll
-            for (int i = 0; i < NPT; i++) {
-                if (BONUS) c[i & 3] = fmaf(S[i], qq[i], c[i & 3]);
-                S[i] = fmaf(gg[i], S[i], kk[i] * w);
-                if (PHASE == 1) P[i] *= gg[i];
-                if (!BONUS) c[i & 3] = fmaf(S[i], qq[i], c[i & 3]);
+            for (int u = 0; u < kScanStep; u++) {
+                acc[u] = 0.f, w[u] = 0.f;
+                if (tt + u < nt) {
+                    float kk[NPT], gg[NPT], c[4] = {0.f, 0.f, 0.f, 0.f};
+                    slice(kk, sK, tt + u, 0.f), decays(gg, tt + u);
+                    w[u] = sV[(tt + u) * PB + pv];
+                    if (emit && BONUS) {
+                        float qq[NPT];
+                        slice(qq, sQ, tt + u, 0.f);
+#pragma unroll
+                        for (int i = 0; i < NPT; i++) c[i & 3] = fmaf(S[i], qq[i], c[i & 3]);
+                    }
+#pragma unroll
+                    for (int i = 0; i < NPT; i++) {
+                        S[i] = fmaf(gg[i], S[i], kk[i] * w[u]);
+                        if (PHASE == 1) P[PHASE == 1 ? i : 0] *= gg[i];
+                    }
+                    if (emit && !BONUS) {
+                        float qq[NPT];
+                        slice(qq, sQ, tt + u, 0.f);
+#pragma unroll
+                        for (int i = 0; i < NPT; i++) c[i & 3] = fmaf(S[i], qq[i], c[i & 3]);
+                    }
+                    acc[u] = (c[0] + c[1]) + (c[2] + c[3]);
+                }
             }
             if (!emit) continue;
-            float acc = (c[0] + c[1]) + (c[2] + c[3]);
-            for (int o = R >> 1; o > 0; o >>= 1) acc += __shfl_xor_sync(0xffffffffu, acc, o);
-            if (live && r == 0) a.y[(size_t)(m0 + t0 + tt) * a.ldy + h * a.dv + p] = BONUS ? fmaf(sKQ[tt], w, acc) : acc;
+            for (int o = R >> 1; o > 0; o >>= 1)
+#pragma unroll
+                for (int u = 0; u < kScanStep; u++) acc[u] += __shfl_xor_sync(0xffffffffu, acc[u], o);
+#pragma unroll
+            for (int u = 0; u < kScanStep; u++)  // the lanes of a column share the stores
+                if (live && tt + u < nt && (u & (R - 1)) == r) yt[(size_t)(tt + u) * a.ldy] = BONUS ? fmaf(sKQ[tt + u], w[u], acc[u]) : acc[u];
         }
     }
     if (!live || (PHASE == 2 && ch != a.nch - 1)) return;
@@ -243,7 +304,7 @@ __global__ void __launch_bounds__(256) kf_gated_scan_kernel(ScanArgs a) {
         float* pr = a.prods + (((size_t)seq * (a.nch - 1) + ch) * a.H + h) * dk;
 #pragma unroll
         for (int i = 0; i < NPT; i++)
-            if (n0 + i < dk) pr[n0 + i] = P[i];
+            if (n0 + i < dk) pr[n0 + i] = P[PHASE == 1 ? i : 0];
     }
 }
 
@@ -477,12 +538,14 @@ static int scan_launch(kf_ctx* ctx, ScanArgs& a, int nseq, int rule) {
     // the decay's exponentials, formed once per CTA) is shared by the CTA's columns -- so columns are NOT spread over more, thinner CTAs
     const int PB = std::max(1, std::min(dv, 256 / R));
     const int threads = std::max(32, ((PB * R + 31) / 32) * 32);
-    const int dkp = ((dk + 15) / 16) * 20;
+    const int dkp = ((dk + 31) / 32) * 36;
     int TB = (int)std::min<size_t>(32, (44 * 1024 / sizeof(float)) / (size_t)(3 * dkp + PB + 2));
     TB = std::max(1, std::min(TB, T));
     const size_t smem = (size_t)(3 * TB * dkp + TB * PB + 2 * TB) * sizeof(float);
     KF_REQUIRE(ctx, smem <= 48 * 1024, "staging area");
     a.R = R, a.PB = PB, a.TB = TB, a.dkp = dkp;
+    a.vec = dk % 4 == 0 && a.ldk % 4 == 0 && a.ldq % 4 == 0 && (a.z_head || a.ldz % 4 == 0) && (((uintptr_t)a.k | (uintptr_t)a.q | (a.z_head ? 0 : (uintptr_t)a.z)) & 15) == 0 &&
+            (((uintptr_t)a.zbias) & 7) == 0;
     const bool full = dk == R * NPT;
     const int cols = (dv + PB - 1) / PB;
     // long panels: chunks of at least 64 tokens, at most 16 of them
