@@ -462,6 +462,10 @@ int kf_attn_window_ex(kf_ctx* ctx, void* out_dev, int out_f32, int ldo, const fl
 int kf_attn_pooled_prefill(kf_ctx* ctx, void* out_bf16_dev, int ldo, const void* q_bf16_dev, const void* cache_dev, size_t slot_stride, int ring,
                            const void* sink_bf16_dev, const int32_t* pos_dev, const int32_t* slot_dev, int M, int n_head, int n_kv, int hd, float scale,
                            float softcap, int window, int pool, const float* head_gate_dev, int ldg, float out_scale);
+/* kf_attn_window_prefill with values of their own size (dk 64 or 128, dv 32, 64 or 128; cache rows [n_kv * dk | n_kv * dv]) */
+int kf_attn_window_prefill_ex(kf_ctx* ctx, void* out_bf16_dev, int ldo, const void* q_bf16_dev, const void* cache_dev, size_t slot_stride, int ring,
+                              const void* sink_bf16_dev, const int32_t* pos_dev, const int32_t* slot_dev, int M, int n_head, int n_kv, int dk, int dv, float scale,
+                              float softcap, int window, float out_scale);
 /* ---- stacks whose norm is n(x) = tanh(alpha x) w + b, entry by entry ----
  * One step of the residual stream: x = res + scale * (what the call adds), out = n(x) in the activation type. */
 typedef struct kf_dyt_step {

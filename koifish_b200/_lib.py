@@ -157,6 +157,7 @@ SIGNATURES = {
     "kf_qk_heads_prepare": (_I, [_P, _P, _I, _I, _I, _I, _I, _P, _P, _F, _I, _P, _F, _I, _P, _I, _SZ, _I, _I, _I, _P, _P, _P, _I]),
     "kf_attn_window_ex": (_I, [_P, _P, _I, _I, _P, _I, _P, _I, _SZ, _I, _P, _P, _P, _I, _I, _I, _I, _I, _F, _F, _I, _I, _F, _I, _P, _I]),
     "kf_attn_pooled_prefill": (_I, [_P, _P, _I, _P, _P, _SZ, _I, _P, _P, _P, _I, _I, _I, _I, _F, _F, _I, _I, _P, _I, _F]),
+    "kf_attn_window_prefill_ex": (_I, [_P, _P, _I, _P, _P, _SZ, _I, _P, _P, _P, _I, _I, _I, _I, _I, _F, _F, _I, _F]),
     "kf_dyt_residual": (_I, [_P, C.POINTER(DytStep), _P, _I]),
     "kf_dyt_experts": (_I, [_P, C.POINTER(DytStep), _P, _P, _P, _P, _I]),
     "kf_dyt_embed": (_I, [_P, C.POINTER(DytStep), _DESCP, _P]),

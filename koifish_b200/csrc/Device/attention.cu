@@ -575,13 +575,13 @@ struct PfBias {
 // softmax weights of MODE 1 without penalty and gate, with the window, cap, sink and ring of PfBias.  MODE 3: the rows and the ring of
 // MODE 2 with sigmoid weights inside blocks of positions -- no running maximum, no rescaling, no denominator.  MODE 4: MODE 2 over pooled
 // blocks as well, whose tiles come ahead of the window's.
-template <int HD, int BKV, int MODE>
+template <int HD, int BKV, int MODE, int VD = HD>
 __global__ void __launch_bounds__(128, KF_PF_MINB) kf_attn_prefill_kernel(uint16_t* __restrict__ out, const uint16_t* __restrict__ q,
                                                               const uint16_t* __restrict__ kc, const uint16_t* __restrict__ vc,
                                                               const int32_t* __restrict__ pos_dev, int M, int n_head, int n_kv, int max_seq,
                                                               float sqrt_hd, PfBias xb) {
     constexpr bool BIAS = MODE == 1, WIN = MODE == 2 || MODE == 4, SIG = MODE == 3, POOL = MODE == 4, RING = MODE >= 2, ROWS = MODE != 0;
-    constexpr int CH = HD / 8;  // 16-byte chunks per row
+    constexpr int CH = HD / 8, CHV = VD / 8;  // 16-byte chunks per row
     extern __shared__ __align__(16) uint8_t pf_smem[];
     const uint32_t sQ = (uint32_t)__cvta_generic_to_shared(pf_smem);
     const uint32_t sK = sQ + kPfQ * HD * 2;            // two K tiles
@@ -604,6 +604,8 @@ __global__ void __launch_bounds__(128, KF_PF_MINB) kf_attn_prefill_kernel(uint16
     const int b_lo = SIG ? ((pos0 + q0 + (threadIdx.x >> 5) * 16 + ((threadIdx.x & 31) >> 2)) / xb.block) * xb.block : 0;
     const int b_hi = SIG ? ((pos0 + q0 + (threadIdx.x >> 5) * 16 + ((threadIdx.x & 31) >> 2) + 8) / xb.block) * xb.block : 0;
     auto sw = [](int row, int c) { return (uint32_t)((row * CH + (c ^ (row & 7))) * 16); };
+    // rows of four chunks: two rows share a 128-byte line, the pair's number permutes the chunks
+    auto swv = [](int row, int c) { return (uint32_t)((row * CHV + (CHV >= 8 ? c ^ (row & 7) : c ^ ((row >> 1) & 3))) * 16); };
 
     // ---- Q tile + first K / V tile ----
     for (int i = tid; i < kPfQ * CH; i += 128) {
@@ -613,9 +615,8 @@ __global__ void __launch_bounds__(128, KF_PF_MINB) kf_attn_prefill_kernel(uint16
     }
     auto load_kv = [&](int kt, int buf) {
         const int tb = RING ? max(kt, 0) * BKV % xb.ring : 0;
-        for (int i = tid; i < BKV * CH; i += 128) {
-            const int r = i / CH, c = i % CH;
-            // rows past kv_len are masked below; keep the address inside the cache (WIN: any row of the ring will do for those)
+        // rows past kv_len are masked below; keep the address inside the cache (WIN: any row of the ring will do for those)
+        auto row_of = [&](int r) {
             int t;
             if (POOL && kt < kt0) {
                 t = xb.ring + min((kt - it0) * BKV + r, nb_max - 1);
@@ -625,17 +626,27 @@ __global__ void __launch_bounds__(128, KF_PF_MINB) kf_attn_prefill_kernel(uint16
             } else {
                 t = min(kt * BKV + r, max_seq - 1);
             }
-            cp16(sK + buf * (BKV * HD * 2) + sw(r, c), kc + (size_t)t * kv_dim + (size_t)kvh * HD + c * 8, true);
-            cp16(sV + buf * (BKV * HD * 2) + sw(r, c), vc + (size_t)t * kv_dim + (size_t)kvh * HD + c * 8, true);
+            return (size_t)t * kv_dim;
+        };
+        for (int i = tid; i < BKV * CH; i += 128) {
+            const int r = i / CH, c = i % CH;
+            const size_t row = row_of(r);
+            cp16(sK + buf * (BKV * HD * 2) + sw(r, c), kc + row + (size_t)kvh * HD + c * 8, true);
+            if (VD == HD) cp16(sV + buf * (BKV * VD * 2) + swv(r, c), vc + row + (size_t)kvh * VD + c * 8, true);
         }
+        if (VD != HD)
+            for (int i = tid; i < BKV * CHV; i += 128) {
+                const int r = i / CHV, c = i % CHV;
+                cp16(sV + buf * (BKV * VD * 2) + swv(r, c), vc + row_of(r) + (size_t)kvh * VD + c * 8, true);
+            }
     };
     load_kv(it0, it0 & 1);
     asm volatile("cp.async.commit_group;" ::: "memory");
 
     uint32_t qa[HD / 16][4];
-    float o[HD / 8][4];
+    float o[VD / 8][4];
 #pragma unroll
-    for (int j = 0; j < HD / 8; j++) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
+    for (int j = 0; j < VD / 8; j++) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
     float m_lo = -INFINITY, m_hi = -INFINITY, l_lo = 0.f, l_hi = 0.f;
     const int p_lo = pos0 + q0 + warp * 16 + g, p_hi = p_lo + 8;  // positions of this thread's two query rows
     // softmax((q.k)/sqrt(hd)) = 2^((q.k - max) * log2(e)/sqrt(hd)) / sum ; BIAS: the scores are brought to the log2 domain where the penalty joins
@@ -652,7 +663,7 @@ __global__ void __launch_bounds__(128, KF_PF_MINB) kf_attn_prefill_kernel(uint16
 #pragma unroll
             for (int kc_ = 0; kc_ < HD / 16; kc_++) ldsm_x4(qa[kc_], sQ + sw(warp * 16 + (lane & 15), kc_ * 2 + (lane >> 4)));
         }
-        const uint32_t kb = sK + buf * (BKV * HD * 2), vb = sV + buf * (BKV * HD * 2);
+        const uint32_t kb = sK + buf * (BKV * HD * 2), vb = sV + buf * (BKV * VD * 2);
         // ---- S = Q K^T (16 x 64 per warp) ----
         float sc[BKV / 8][4];
 #pragma unroll
@@ -738,15 +749,15 @@ __global__ void __launch_bounds__(128, KF_PF_MINB) kf_attn_prefill_kernel(uint16
         l_lo = l_lo * c_lo + rs_lo, l_hi = l_hi * c_hi + rs_hi;
         if (!SIG) {
 #pragma unroll
-            for (int j = 0; j < HD / 8; j++) o[j][0] *= c_lo, o[j][1] *= c_lo, o[j][2] *= c_hi, o[j][3] *= c_hi;
+            for (int j = 0; j < VD / 8; j++) o[j][0] *= c_lo, o[j][1] *= c_lo, o[j][2] *= c_hi, o[j][3] *= c_hi;
         }
         // ---- O += P V ----
 #pragma unroll
         for (int kc_ = 0; kc_ < BKV / 16; kc_++) {
 #pragma unroll
-            for (int jp = 0; jp < HD / 16; jp++) {
+            for (int jp = 0; jp < VD / 16; jp++) {
                 uint32_t b[4];
-                ldsm_x4_t(b, vb + sw(kc_ * 16 + (lane & 7) + ((lane >> 3) & 1) * 8, jp * 2 + (lane >> 4)));
+                ldsm_x4_t(b, vb + swv(kc_ * 16 + (lane & 7) + ((lane >> 3) & 1) * 8, jp * 2 + (lane >> 4)));
                 mma_bf16(o[2 * jp], pa[kc_], b[0], b[1]);
                 mma_bf16(o[2 * jp + 1], pa[kc_], b[2], b[3]);
                 if (ROWS) {
@@ -766,16 +777,16 @@ __global__ void __launch_bounds__(128, KF_PF_MINB) kf_attn_prefill_kernel(uint16
         const float c_lo = exp2f(m_lo - n_lo), c_hi = exp2f(m_hi - n_hi);
         l_lo = l_lo * c_lo + exp2f(s2 - n_lo), l_hi = l_hi * c_hi + exp2f(s2 - n_hi);
 #pragma unroll
-        for (int j = 0; j < HD / 8; j++) o[j][0] *= c_lo, o[j][1] *= c_lo, o[j][2] *= c_hi, o[j][3] *= c_hi;
+        for (int j = 0; j < VD / 8; j++) o[j][0] *= c_lo, o[j][1] *= c_lo, o[j][2] *= c_hi, o[j][3] *= c_hi;
     }
     float i_lo = SIG ? xb.out_scale : (WIN ? xb.out_scale : 1.f) / l_lo, i_hi = SIG ? xb.out_scale : (WIN ? xb.out_scale : 1.f) / l_hi;
-    const int r_lo = q0 + warp * 16 + g, r_hi = r_lo + 8, o_dim = RING ? xb.out_ld : q_dim;
+    const int r_lo = q0 + warp * 16 + g, r_hi = r_lo + 8, o_dim = RING ? xb.out_ld : n_head * VD;
     if (POOL && xb.hgate) {
         if (r_lo < M) i_lo *= 1.f / (1.f + expf(-xb.hgate[(size_t)r_lo * xb.ldg + h]));
         if (r_hi < M) i_hi *= 1.f / (1.f + expf(-xb.hgate[(size_t)r_hi * xb.ldg + h]));
     }
 #pragma unroll
-    for (int j = 0; j < HD / 8; j++) {
+    for (int j = 0; j < VD / 8; j++) {
         const int d = j * 8 + 2 * t4;
         float g0 = 1.f, g1 = 1.f, g2 = 1.f, g3 = 1.f;
         if (BIAS && xb.gate) {
@@ -788,8 +799,8 @@ __global__ void __launch_bounds__(128, KF_PF_MINB) kf_attn_prefill_kernel(uint16
                 g2 = 1.f / (1.f + expf(-z.x)), g3 = 1.f / (1.f + expf(-z.y));
             }
         }
-        if (r_lo < M) *reinterpret_cast<uint32_t*>(out + (size_t)r_lo * o_dim + (size_t)h * HD + d) = pack_bf16x2(o[j][0] * i_lo * g0, o[j][1] * i_lo * g1);
-        if (r_hi < M) *reinterpret_cast<uint32_t*>(out + (size_t)r_hi * o_dim + (size_t)h * HD + d) = pack_bf16x2(o[j][2] * i_hi * g2, o[j][3] * i_hi * g3);
+        if (r_lo < M) *reinterpret_cast<uint32_t*>(out + (size_t)r_lo * o_dim + (size_t)h * VD + d) = pack_bf16x2(o[j][0] * i_lo * g0, o[j][1] * i_lo * g1);
+        if (r_hi < M) *reinterpret_cast<uint32_t*>(out + (size_t)r_hi * o_dim + (size_t)h * VD + d) = pack_bf16x2(o[j][2] * i_hi * g2, o[j][3] * i_hi * g3);
     }
 }
 
@@ -1151,34 +1162,43 @@ extern "C" int kf_attn_bias_prefill(kf_ctx* ctx, void* out, const void* q_bf16, 
 extern "C" int kf_attn_window_prefill(kf_ctx* ctx, void* out, int ldo, const void* q_bf16, const void* cache, size_t slot_stride, int ring, const void* sink_bf16,
                                       const int32_t* pos_dev, const int32_t* slot_dev, int M, int n_head, int n_kv, int hd, float scale, float softcap,
                                       int window, float out_scale) {
-    if (!ctx || !out || !q_bf16 || !cache || !pos_dev || !slot_dev) return KF_ERR_BAD_ARG;
-    KF_REQUIRE(ctx, (hd == 128 || hd == 64) && n_head % n_kv == 0 && M >= 1 && ring >= 1 && (window <= 0 || ring >= window) && ldo >= n_head * hd && ldo % 2 == 0,
-               "head size 64/128, GQA, ring");
-    const size_t smem = (size_t)(kPfQ + 4 * KF_PF_BKV) * hd * 2;
-    dim3 grid((M + kPfQ - 1) / kPfQ, n_head);
-    PfBias xb = {nullptr, nullptr, nullptr, 0, slot_dev, slot_stride, 2 * n_kv * hd, scale, ring, window > 0 ? window : 0x3fffffff, softcap,
-                 (const uint16_t*)sink_bf16, ldo, out_scale};
-    const uint16_t* kc = (const uint16_t*)cache;
-    const uint16_t* vc = kc + (size_t)n_kv * hd;
-    if (hd == 128) {
-        static bool set[kf_ctx::kMaxDevices] = {};
-        if (!set[ctx->device]) {
-            KF_CUDA(ctx, cudaFuncSetAttribute(kf_attn_prefill_kernel<128, KF_PF_BKV, 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-            set[ctx->device] = true;
-        }
-        kf_attn_prefill_kernel<128, KF_PF_BKV, 2><<<grid, 128, smem, ctx->stream>>>((uint16_t*)out, (const uint16_t*)q_bf16, kc, vc, pos_dev, M, n_head, n_kv, ring,
-                                                                                  1.f, xb);
-    } else {
-        static bool set[kf_ctx::kMaxDevices] = {};
-        if (!set[ctx->device]) {
-            KF_CUDA(ctx, cudaFuncSetAttribute(kf_attn_prefill_kernel<64, KF_PF_BKV, 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-            set[ctx->device] = true;
-        }
-        kf_attn_prefill_kernel<64, KF_PF_BKV, 2><<<grid, 128, smem, ctx->stream>>>((uint16_t*)out, (const uint16_t*)q_bf16, kc, vc, pos_dev, M, n_head, n_kv, ring,
-                                                                                 1.f, xb);
+    return kf_attn_window_prefill_ex(ctx, out, ldo, q_bf16, cache, slot_stride, ring, sink_bf16, pos_dev, slot_dev, M, n_head, n_kv, hd, hd, scale, softcap, window, out_scale);
+}
+template <int HD, int VD>
+static int window_prefill(kf_ctx* ctx, void* out, const void* q, const uint16_t* cache, const int32_t* pos, int M, int n_head, int n_kv, int ring, const PfBias& xb) {
+    const size_t smem = (size_t)(kPfQ * HD + 2 * KF_PF_BKV * (HD + VD)) * 2;
+    static bool set[kf_ctx::kMaxDevices] = {};
+    if (!set[ctx->device]) {
+        KF_CUDA(ctx, cudaFuncSetAttribute(kf_attn_prefill_kernel<HD, KF_PF_BKV, 2, VD>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+        set[ctx->device] = true;
     }
+    kf_attn_prefill_kernel<HD, KF_PF_BKV, 2, VD><<<dim3((M + kPfQ - 1) / kPfQ, n_head), 128, smem, ctx->stream>>>((uint16_t*)out, (const uint16_t*)q, cache,
+                                                                                                                cache + (size_t)n_kv * HD, pos, M, n_head, n_kv, ring, 1.f, xb);
     KF_LAUNCH_CHECK(ctx);
     return KF_OK;
+}
+// The same with values of their own size: cache rows [n_kv * dk keys | n_kv * dv values], dk 64 or 128, dv 32, 64 or 128; out [M][ldo] has n_head * dv
+// entries per row.
+extern "C" int kf_attn_window_prefill_ex(kf_ctx* ctx, void* out, int ldo, const void* q_bf16, const void* cache, size_t slot_stride, int ring, const void* sink_bf16,
+                                         const int32_t* pos_dev, const int32_t* slot_dev, int M, int n_head, int n_kv, int dk, int dv, float scale, float softcap,
+                                         int window, float out_scale) {
+    if (!ctx || !out || !q_bf16 || !cache || !pos_dev || !slot_dev) return KF_ERR_BAD_ARG;
+    KF_REQUIRE(ctx, (dk == 128 || dk == 64) && (dv == 128 || dv == 64 || dv == 32) && n_kv >= 1 && n_head % n_kv == 0 && M >= 1 && ring >= 1 &&
+                        (window <= 0 || ring >= window) && ldo >= n_head * dv && ldo % 2 == 0 && slot_stride % 8 == 0 && (((uintptr_t)cache | (uintptr_t)q_bf16) & 15) == 0,
+               "key size 64/128, value size 32/64/128, GQA, ring, 16-byte aligned rows");
+    PfBias xb = {nullptr, nullptr, nullptr, 0, slot_dev, slot_stride, n_kv * (dk + dv), scale, ring, window > 0 ? window : 0x3fffffff, softcap,
+                 (const uint16_t*)sink_bf16, ldo, out_scale};
+    const uint16_t* c = (const uint16_t*)cache;
+#define KF_WP(K, V) \
+    if (dk == K && dv == V) return window_prefill<K, V>(ctx, out, q_bf16, c, pos_dev, M, n_head, n_kv, ring, xb)
+    KF_WP(128, 128);
+    KF_WP(128, 64);
+    KF_WP(128, 32);
+    KF_WP(64, 128);
+    KF_WP(64, 64);
+    KF_WP(64, 32);
+#undef KF_WP
+    return KF_ERR_BAD_ARG;
 }
 
 // kf_attn_window_ex for a panel of M consecutive tokens of one slot on the tensor cores: kf_attn_window_prefill with mean rows of blocks of

@@ -50,7 +50,7 @@ struct ScanArgs {
 // (normalised there), the decay (formed there), v, beta.  FULL (dk == R * NPT): a thread's slice of k, q and the decay is NPT / 4 16-byte
 // shared loads each and nothing is bounds-checked; otherwise rows beyond dk read k = q = 0 and leave their (zero) state alone.
 constexpr int NPT_MAX = 16;
-constexpr int kScanChunk = 64;
+constexpr int kScanChunk = 32;
 constexpr int kScanStep = 4;  // rules 0 and 2: read-outs of this many tokens are reduced over the lanes together
 // RULE 0: plain outer-product write; 1: delta-rule write; 2: read-out ahead of the write, with a bonus.
 // PHASE 0: a CTA walks all T tokens.  Long panels of the rules whose state map is affine with a diagonal factor (0 and 2) go in two launches over
@@ -87,6 +87,7 @@ __global__ void __launch_bounds__(256, NPT == 8 ? 3 : 2) kf_gated_scan_kernel(Sc
         const float* q0 = a.prods + (size_t)seq * (a.nch - 1) * ps + (size_t)h * dk;
 #pragma unroll
         for (int i = 0; i < NPT; i++) S[i] = (live && n0 + i < dk) ? e0[n0 + i] : 0.f;
+#pragma unroll 2
         for (int j = 1; j < ch; j++) {
 #pragma unroll
             for (int i = 0; i < NPT; i++)
@@ -306,6 +307,93 @@ __global__ void __launch_bounds__(256, NPT == 8 ? 3 : 2) kf_gated_scan_kernel(Sc
         for (int i = 0; i < NPT; i++)
             if (n0 + i < dk) pr[n0 + i] = P[PHASE == 1 ? i : 0];
     }
+}
+
+// One token per sequence (decoding): the same update without staging -- a thread fetches its slices of k, q, the decay logits and the state
+// itself, all at once, and forms its decays; a column's lanes add up the token's sums by shuffles.  Rows beyond dk count as zeros.
+template <int RULE, int NPT>
+__global__ void __launch_bounds__(128) kf_gated_scan_one_kernel(ScanArgs a) {
+    constexpr bool DELTA = RULE == 1, BONUS = RULE == 2;
+    const int h = blockIdx.x, m = blockIdx.y, dk = a.dk, R = a.R;
+    const int kh = h / (a.H / a.G), pl = threadIdx.x / R, r = threadIdx.x - pl * R, p = blockIdx.z * a.PB + pl, n0 = r * NPT;
+    const bool live = pl < a.PB && p < a.dv;
+    float* st = a.state + (size_t)a.slot[m] * a.state_stride + ((size_t)h * a.dv + (live ? p : 0)) * dk;
+    const bool fresh = a.pos[m] == 0;
+    float S[NPT], kk[NPT], qq[NPT], gg[NPT], uu[NPT];
+    auto rows = [&](float (&to)[NPT], const float* from) {
+#pragma unroll
+        for (int i = 0; i < NPT; i += 4) {
+            if (a.vec) {
+                const float4 f = n0 + i < dk ? *reinterpret_cast<const float4*>(from + n0 + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+                to[i] = f.x, to[i + 1] = f.y, to[i + 2] = f.z, to[i + 3] = f.w;
+            } else {
+#pragma unroll
+                for (int e = 0; e < 4; e++) to[i + e] = n0 + i + e < dk ? from[n0 + i + e] : 0.f;
+            }
+        }
+    };
+    auto halves = [&](float (&to)[NPT], const uint16_t* from) {
+#pragma unroll
+        for (int i = 0; i < NPT; i++) to[i] = n0 + i < dk ? bf16_bits_to_f32(from[n0 + i]) : 0.f;
+    };
+    rows(kk, a.k + (size_t)m * a.ldk + kh * dk), rows(qq, a.q + (size_t)m * a.ldq + kh * dk);
+    if (!a.z_head) rows(gg, a.z + (size_t)m * a.ldz + h * dk);
+#pragma unroll
+    for (int i = 0; i < NPT; i++) S[i] = (live && n0 + i < dk) ? st[n0 + i] : 0.f;
+    if (fresh)
+#pragma unroll
+        for (int i = 0; i < NPT; i++) S[i] = 0.f;
+    if (BONUS) halves(uu, a.bonus + h * dk);
+    const float v = live ? a.v[(size_t)m * a.ldv + h * a.dv + p] : 0.f, beta = DELTA ? sigmoid_f(a.beta[(size_t)m * a.ldb + h]) : 0.f;
+    const float Aexp = a.decay_kind == 1 ? expf(bf16_bits_to_f32(a.A_log[h])) : 0.f;
+    auto decay = [&](float z) {
+        return a.decay_kind == 2 ? expf(-expf(z)) : a.decay_kind == 1 ? expf(-Aexp * softplus_f(z)) : expf(log_sigmoid_f(z) * a.inv_tau);
+    };
+    if (a.z_head) {
+        const float g = decay(a.z[(size_t)m * a.ldz + h] + (a.zbias ? bf16_bits_to_f32(a.zbias[h]) : 0.f));
+#pragma unroll
+        for (int i = 0; i < NPT; i++) gg[i] = g;
+    } else {
+        if (a.zbias) {
+            float b[NPT];
+            halves(b, a.zbias + h * dk);
+#pragma unroll
+            for (int i = 0; i < NPT; i++) gg[i] += b[i];
+        }
+#pragma unroll
+        for (int i = 0; i < NPT; i++) gg[i] = decay(gg[i]);
+    }
+    if (a.unit_qk) {
+        float sq = 0.f, sk = 0.f;
+#pragma unroll
+        for (int i = 0; i < NPT; i++) sq = fmaf(qq[i], qq[i], sq), sk = fmaf(kk[i], kk[i], sk);
+        for (int o = R >> 1; o > 0; o >>= 1) sq += __shfl_xor_sync(0xffffffffu, sq, o), sk += __shfl_xor_sync(0xffffffffu, sk, o);
+        const float fq = 1.f / sqrtf(sq + a.unit_eps), fk = 1.f / sqrtf(sk + a.unit_eps);
+#pragma unroll
+        for (int i = 0; i < NPT; i++) qq[i] *= fq, kk[i] *= fk;
+    }
+    // sums over the key channels: the read-out of the state (decayed, except ahead of the write), k . q (or (u * k) . q), the state along k
+    float rd[2] = {0.f, 0.f}, kq[2] = {0.f, 0.f}, dot[2] = {0.f, 0.f};
+#pragma unroll
+    for (int i = 0; i < NPT; i++) {
+        qq[i] *= a.q_scale;
+        if (BONUS) rd[i & 1] = fmaf(S[i], qq[i], rd[i & 1]);
+        S[i] *= gg[i];
+        if (!BONUS) rd[i & 1] = fmaf(S[i], qq[i], rd[i & 1]);
+        if (DELTA) dot[i & 1] = fmaf(S[i], kk[i], dot[i & 1]);
+        kq[i & 1] = fmaf(BONUS ? uu[i] * kk[i] : kk[i], qq[i], kq[i & 1]);
+    }
+    float c0 = rd[0] + rd[1], c1 = kq[0] + kq[1], c2 = dot[0] + dot[1];
+    for (int o = R >> 1; o > 0; o >>= 1) {
+        c0 += __shfl_xor_sync(0xffffffffu, c0, o), c1 += __shfl_xor_sync(0xffffffffu, c1, o);
+        if (DELTA) c2 += __shfl_xor_sync(0xffffffffu, c2, o);
+    }
+    const float w = DELTA ? beta * (v - c2) : v;
+    if (!live) return;
+#pragma unroll
+    for (int i = 0; i < NPT; i++)
+        if (n0 + i < dk) st[n0 + i] = fmaf(kk[i], w, S[i]);
+    if (r == 0) a.y[(size_t)m * a.ldy + h * a.dv + p] = fmaf(c1, w, c0);
 }
 
 // ------------------------------------------------------------------------------------------------------------ real-gated LRU
@@ -546,10 +634,23 @@ static int scan_launch(kf_ctx* ctx, ScanArgs& a, int nseq, int rule) {
     a.R = R, a.PB = PB, a.TB = TB, a.dkp = dkp;
     a.vec = dk % 4 == 0 && a.ldk % 4 == 0 && a.ldq % 4 == 0 && (a.z_head || a.ldz % 4 == 0) && (((uintptr_t)a.k | (uintptr_t)a.q | (a.z_head ? 0 : (uintptr_t)a.z)) & 15) == 0 &&
             (((uintptr_t)a.zbias) & 7) == 0;
+    if (T == 1) {
+        a.PB = std::max(1, std::min(dv, 128 / R));
+        const dim3 g1(H, nseq, (dv + a.PB - 1) / a.PB);
+        const int th = std::max(32, ((a.PB * R + 31) / 32) * 32);
+#define KF_ONE(D) (NPT == 8 ? kf_gated_scan_one_kernel<D, 8><<<g1, th, 0, ctx->stream>>>(a) : kf_gated_scan_one_kernel<D, 16><<<g1, th, 0, ctx->stream>>>(a))
+        if (rule == 1) KF_ONE(1);
+        else if (rule == 2) KF_ONE(2);
+        else KF_ONE(0);
+#undef KF_ONE
+        KF_LAUNCH_CHECK(ctx);
+        return KF_OK;
+    }
     const bool full = dk == R * NPT;
     const int cols = (dv + PB - 1) / PB;
-    // long panels: chunks of at least 64 tokens, at most 16 of them
-    const int nch = rule != 1 && T >= 2 * kScanChunk ? std::min(16, T / kScanChunk) : 1;
+    // long panels: as many chunks of at least kScanChunk tokens as the SMs hold CTAs at once
+    const int room = (NPT == 8 ? 3 : 2) * ctx->sm_count / (H * nseq * cols);
+    const int nch  = rule != 1 && T >= 2 * kScanChunk ? std::min(room + 1, T / kScanChunk) : 1;
     if (nch > 1) {
         a.chunk = (T + nch - 1) / nch, a.nch = (T + a.chunk - 1) / a.chunk;
         const size_t ends = (size_t)nseq * (a.nch - 1) * H * dv * dk, prods = (size_t)nseq * (a.nch - 1) * H * dk;

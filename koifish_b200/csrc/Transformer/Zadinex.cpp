@@ -363,13 +363,13 @@ int BlendedAttention::cuInfer(int M, float* u, int ldu, int layer) {
     SeqStateCache::Layer& sl = f.states.layers[layer];
     const int ring = c.max_seq_len;  // every position keeps its row
     // panels of one sequence with head sizes the tensor-core kernel takes go there; everything else (decode, other sizes, 32-bit) to the general kernel
-    const bool tile = !ak && f.panel_consecutive && f.seq_mode == 0 && M >= 16 && m.dim == m.vdim && (m.dim == 64 || m.dim == 128);
+    const bool tile = !ak && f.panel_consecutive && f.seq_mode == 0 && M >= 16 && (m.dim == 64 || m.dim == 128) && (m.vdim == 32 || m.vdim == 64 || m.vdim == 128);
     KF_TRY(kf_qk_heads_prepare_ex(f.ctx, u, ldu, m.heads, m.kv_heads, m.dim, m.vdim, nullptr, nullptr, 1, c.norm_rms_eps, m.rot_dims, inv_freq, 1.f, 1,
                                   m.v_mix ? s.vfirst : nullptr, m.kv_heads * m.vdim, m.v_mix && !blend_source ? vmix->data : nullptr, sl.rows, ak, sl.row_stride, ring, 0,
                                   f.seq_mode || M == 1, tile ? s.y : nullptr, f.d_pos, f.d_slot, M));
     if (tile)
-        KF_TRY(kf_attn_window_prefill(f.ctx, s.act, no, s.y, sl.rows, sl.row_stride, ring, sink->data, f.d_pos, f.d_slot, M, m.heads, m.kv_heads, m.dim, m.scale, 0.f, 0,
-                                      1.f));
+        KF_TRY(kf_attn_window_prefill_ex(f.ctx, s.act, no, s.y, sl.rows, sl.row_stride, ring, sink->data, f.d_pos, f.d_slot, M, m.heads, m.kv_heads, m.dim, m.vdim, m.scale,
+                                         0.f, 0, 1.f));
     else
         KF_TRY(kf_attn_window(f.ctx, s.act, ak, no, u, ldu, sl.rows, ak, sl.row_stride, ring, sink->data, f.d_pos, f.d_slot, M, m.heads, m.kv_heads, m.dim, m.vdim,
                               m.scale, 0.f, 0, f.attn_hint + 1, 1.f));
