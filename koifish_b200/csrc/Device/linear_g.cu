@@ -339,6 +339,13 @@ __global__ void __launch_bounds__(256) kf_lin_tile_kernel(LinArgs a) {
                 }
             }
         } else {
+            // a step's products are summed on their own and then added: the rounding error grows with K / BK + BK terms, not with K
+            float p0[16], p1[DUAL ? 16 : 1];
+#pragma unroll
+            for (int i = 0; i < 16; i++) p0[i] = 0.f;
+            if (DUAL)
+#pragma unroll
+                for (int i = 0; i < 16; i++) p1[DUAL ? i : 0] = 0.f;
 #pragma unroll 8
             for (int k = 0; k < BK; k++) {
                 float xv[4], wv[4], uv[4];
@@ -353,10 +360,15 @@ __global__ void __launch_bounds__(256) kf_lin_tile_kernel(LinArgs a) {
                 for (int i = 0; i < 4; i++)
 #pragma unroll
                     for (int j = 0; j < 4; j++) {
-                        acc0[i * 4 + j] = fmaf(xv[i], wv[j], acc0[i * 4 + j]);
-                        if (DUAL) acc1[i * 4 + j] = fmaf(xv[i], uv[j], acc1[i * 4 + j]);
+                        p0[i * 4 + j] = fmaf(xv[i], wv[j], p0[i * 4 + j]);
+                        if (DUAL) p1[DUAL ? i * 4 + j : 0] = fmaf(xv[i], uv[j], p1[DUAL ? i * 4 + j : 0]);
                     }
             }
+#pragma unroll
+            for (int i = 0; i < 16; i++) acc0[i] += p0[i];
+            if (DUAL)
+#pragma unroll
+                for (int i = 0; i < 16; i++) acc1[DUAL ? i : 0] += p1[DUAL ? i : 0];
         }
     }
     auto store = [&](int r, int n, float v0, float v1) {
