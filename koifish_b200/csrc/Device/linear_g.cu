@@ -70,6 +70,7 @@ __global__ void __launch_bounds__(256) kf_lin_gemv_kernel(LinArgs a) {
     float s0 = 0.f, s1 = 0.f;
     const bool vec = (a.K % 8 == 0) && (a.ldx % 8 == 0) && (((uintptr_t)w0 & 15) == 0) && (((uintptr_t)x & 15) == 0) && (!DUAL || ((uintptr_t)w1 & 15) == 0);
     if (vec) {
+#pragma unroll DUAL ? 2 : 4
         for (int k = lane * 8; k < a.K; k += 256) {
             const uint4 wv = *reinterpret_cast<const uint4*>(w0 + k);
             const uint32_t wq[4] = {wv.x, wv.y, wv.z, wv.w};
@@ -439,8 +440,11 @@ extern "C" int kf_linear_g(kf_ctx* ctx, float* y, int ldy, const kf_tensor_desc*
     KF_REQUIRE(ctx, w->type == KF_T_BF16 && M >= 1 && w->rows >= 1 && w->cols >= 1 && ldx >= w->cols && ldy >= w->rows, "bf16 weight, ld >= extent");
     LinArgs a = {};
     a.W0 = (const uint16_t*)w->data_dev, a.x = x, a.y = y, a.M = M, a.N = w->rows, a.K = w->cols, a.ldx = ldx, a.ldy = ldy;
+    // a few rows over a small weight: the warp-per-output kernel is through before the tuned ones have filled their pipelines (measured: 2.9 against
+    // 5.3 us at 1024 x 1024, 4.5 against 6.0 at 2048 x 2048, even at 34 MB of weight x rows)
+    const bool few = M <= kGemvMaxSlots && w->cols <= 4096 && (size_t)M * w->rows * w->cols * 2 <= ((size_t)34 << 20);
     // shapes the tuned kernels take go there (tcgen05 / TMEM panels, the HBM-rate GEMV); fp32 result through their fp32 epilogue
-    if (!skinny_shape(a) && !act_f32 && ldx == w->cols && ldy == w->rows && w->cols % 128 == 0 && w->rows % 16 == 0 && w->rows >= 16 && ctx->tc_min_m != 0 &&
+    if (!few && !skinny_shape(a) && !act_f32 && ldx == w->cols && ldy == w->rows && w->cols % 128 == 0 && w->rows % 16 == 0 && w->rows >= 16 && ctx->tc_min_m != 0 &&
         (((uintptr_t)w->data_dev | (uintptr_t)x | (uintptr_t)y) & 15) == 0)
         return kf_linear(ctx, y, w, x, M, KF_EPI_F32, nullptr);
     return dispatch_one(ctx, a, act_f32);

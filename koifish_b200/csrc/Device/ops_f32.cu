@@ -591,8 +591,14 @@ __device__ __forceinline__ unsigned route_key(float v) {  // unsigned order = fl
     const unsigned u = __float_as_uint(v);
     return (u & 0x80000000u) ? ~u : u | 0x80000000u;
 }
-template <bool CACHED>
-__device__ __forceinline__ void route_grouped_body(int* taken, int32_t* idx, float* __restrict__ wgt, const float* __restrict__ lg,
+// KEEP (CACHED, top <= 32): nothing is written; lane j returns the j-th choice and its weight, every lane the mask of its own outputs taken.
+struct RouteKept {
+    int e;
+    float w;
+    unsigned picked;
+};
+template <bool CACHED, bool KEEP = false>
+__device__ __forceinline__ RouteKept route_grouped_body(int* taken, int32_t* idx, float* __restrict__ wgt, const float* __restrict__ lg,
                                                    const uint16_t* __restrict__ bias, int E, int top, const RouteMode md, int lane) {
     const int per = E / md.groups, n = CACHED ? kRouteCache : (E + 31) / 32;
     float sc[CACHED ? kRouteCache : 1], cv[CACHED ? kRouteCache : 1];
@@ -666,6 +672,7 @@ __device__ __forceinline__ void route_grouped_body(int* taken, int32_t* idx, flo
         }
     }
     float sum = 0.f;
+    RouteKept mine = {0, 0.f, 0u};
     unsigned used = 0;  // CACHED: this lane's outputs that are taken or closed
     if (CACHED) {
 #pragma unroll
@@ -696,16 +703,45 @@ __device__ __forceinline__ void route_grouped_body(int* taken, int32_t* idx, flo
         const int w = (int)min(win, (unsigned)(E - 1));
         if (CACHED) {
             bs = __shfl_sync(0xffffffffu, bs, w & 31);
-            if (lane == (w & 31)) used |= 1u << (w >> 5);
+            if (lane == (w & 31)) used |= 1u << (w >> 5), mine.picked |= 1u << (w >> 5);
         } else {
             bs = score(w);
         }
         sum += bs;
+        if (KEEP) {
+            if (lane == j) mine.e = w, mine.w = md.kind == 2 ? bs : md.scale * bs;
+            continue;
+        }
         if (lane == 0) taken[j] = w, idx[j] = w, wgt[j] = md.kind == 2 ? bs : md.scale * bs;
         __syncwarp();
     }
-    if (md.kind == 2 && lane == 0)
+    if (KEEP && md.kind == 2) mine.w /= sum + 1e-20f;
+    if (!KEEP && md.kind == 2 && lane == 0)
         for (int j = 0; j < top; j++) wgt[j] /= sum + 1e-20f;
+    return mine;
+}
+// One token (decoding) in kinds 1 and 2: choice and dispatch tables by ONE warp without shared memory.  Every expert holds at most one entry, so
+// an entry's slot is the number of chosen experts before its own.
+__global__ void __launch_bounds__(32) kf_moe_route_one_kernel(int32_t* __restrict__ idx, float* __restrict__ wgt, int32_t* __restrict__ offsets,
+                                                              int32_t* __restrict__ entry_slot, int32_t* __restrict__ slot_row, int32_t* __restrict__ slot_group,
+                                                              const float* __restrict__ logits, const uint16_t* __restrict__ bias, int E, int top, const RouteMode md) {
+    const int lane = threadIdx.x, X = E - md.pass;
+    const RouteKept r = route_grouped_body<true, true>(nullptr, nullptr, nullptr, logits, bias, E, top, md, lane);
+    const bool real = lane < top && r.e < X;
+    const int n = __popc(__ballot_sync(0xffffffffu, real));
+    int sl = 0;
+    for (int j = 0; j < top; j++) sl += __shfl_sync(0xffffffffu, r.e, j) < r.e;
+    int before = 0;
+#pragma unroll
+    for (int i = 0; i <= kRouteCache; i++) {
+        const unsigned word = i < kRouteCache ? __ballot_sync(0xffffffffu, (r.picked >> i) & 1u) : 0u;
+        if (32 * i + lane <= X) offsets[32 * i + lane] = before + __popc(word & ((1u << lane) - 1));
+        before += __popc(word);
+    }
+    if (lane >= top) return;
+    idx[lane] = r.e, wgt[lane] = r.w, entry_slot[lane] = real ? sl : -1;
+    if (real) slot_row[sl] = 0, slot_group[sl] = r.e;
+    if (lane >= n) slot_row[lane] = 0, slot_group[lane] = -1;
 }
 __device__ __forceinline__ void route_grouped_warp(int* taken, int32_t* idx, float* __restrict__ wgt, const float* __restrict__ lg,
                                                    const uint16_t* __restrict__ bias, int E, int top, const RouteMode md, int lane) {
@@ -1217,6 +1253,11 @@ static int moe_route_impl(kf_ctx* ctx, int32_t* idx, float* wgt, int32_t* offset
     if (!ctx || !idx || !wgt || !offsets || !entry_slot || !slot_row || !slot_group || !work || !logits) return KF_ERR_BAD_ARG;
     KF_REQUIRE(ctx, M >= 1 && E >= 1 && top >= 1 && top <= E && ldl >= E, "1 <= top <= experts");
     const int n = M * top;
+    if (M == 1 && md.kind && top <= 32 && E <= 32 * kRouteCache) {
+        kf_moe_route_one_kernel<<<1, 32, 0, ctx->stream>>>(idx, wgt, offsets, entry_slot, slot_row, slot_group, logits, (const uint16_t*)bias_bf16, E, top, md);
+        KF_LAUNCH_CHECK(ctx);
+        return KF_OK;
+    }
     if (n <= kRouteSmall && (long long)E * n <= 16384) {
         kf_moe_route_small_kernel<<<1, 256, 0, ctx->stream>>>(idx, wgt, offsets, entry_slot, slot_row, slot_group, logits, ldl, (const uint16_t*)bias_bf16, M, E, top, full_softmax, md);
         KF_LAUNCH_CHECK(ctx);
