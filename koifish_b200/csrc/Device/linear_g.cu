@@ -255,6 +255,62 @@ __device__ __forceinline__ void fetch8(Frag8<T>& f, const T* base, size_t row_of
     for (int j = 0; j < 8; j++) f.v[j] = (row_ok && k + j < K) ? base[row_off + k + j] : T(0);
 }
 
+// The same shapes with bf16 activations on the tensor cores: a CTA takes 16 rows and all outputs (up to 8 * NT), its 8 warps deal the k chunks of
+// 32 among themselves and their sums meet in shared memory, always in the same order.  Fragments come straight from memory: a product over k
+// does not mind how k is numbered, so lane (g, t) of an operand's row g loads the 8 consecutive k 8t .. 8t + 7 of a chunk in one access and
+// hands them out as the k places that two m16n8k16 steps expect of it; both operands use the same numbering.
+template <int NT>
+__global__ void __launch_bounds__(256) kf_lin_skinny_mma_kernel(LinArgs a) {
+    __shared__ __align__(16) float part[4][16][NT * 8 + 2];
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3, m0 = blockIdx.x * 16;
+    const uint16_t* xa = (const uint16_t*)a.x + (size_t)min(m0 + g, a.M - 1) * a.ldx + 8 * t;
+    const uint16_t* xb = (const uint16_t*)a.x + (size_t)min(m0 + g + 8, a.M - 1) * a.ldx + 8 * t;
+    const uint16_t* w[NT];
+#pragma unroll
+    for (int j = 0; j < NT; j++) w[j] = a.W0 + (size_t)min(j * 8 + g, a.N - 1) * a.K + 8 * t;
+    float acc[NT][4];
+#pragma unroll
+    for (int j = 0; j < NT; j++) acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.f;
+    for (int k = warp * 32; k < a.K; k += 256) {
+        const uint4 pa = *reinterpret_cast<const uint4*>(xa + k), pb = *reinterpret_cast<const uint4*>(xb + k);
+        uint4 q[NT];
+#pragma unroll
+        for (int j = 0; j < NT; j++) q[j] = *reinterpret_cast<const uint4*>(w[j] + k);
+        const uint32_t a0[4] = {pa.x, pb.x, pa.y, pb.y}, a1[4] = {pa.z, pb.z, pa.w, pb.w};
+#pragma unroll
+        for (int j = 0; j < NT; j++) {
+            const uint32_t b0[2] = {q[j].x, q[j].y}, b1[2] = {q[j].z, q[j].w};
+            mma_bf16_16816(acc[j], a0, b0);
+            mma_bf16_16816(acc[j], a1, b1);
+        }
+    }
+    auto put = [&](int slot) {
+#pragma unroll
+        for (int j = 0; j < NT; j++) {
+            part[slot][g][j * 8 + 2 * t] = acc[j][0], part[slot][g][j * 8 + 2 * t + 1] = acc[j][1];
+            part[slot][g + 8][j * 8 + 2 * t] = acc[j][2], part[slot][g + 8][j * 8 + 2 * t + 1] = acc[j][3];
+        }
+    };
+    if (warp >= 4) put(warp - 4);
+    __syncthreads();
+    if (warp < 4) {
+#pragma unroll
+        for (int j = 0; j < NT; j++) {
+            acc[j][0] += part[warp][g][j * 8 + 2 * t], acc[j][1] += part[warp][g][j * 8 + 2 * t + 1];
+            acc[j][2] += part[warp][g + 8][j * 8 + 2 * t], acc[j][3] += part[warp][g + 8][j * 8 + 2 * t + 1];
+        }
+        put(warp);  // the places this thread has just read
+    }
+    __syncthreads();
+    for (int i = threadIdx.x; i < 16 * a.N; i += blockDim.x) {
+        const int r = i / a.N, n = i - r * a.N;
+        if (m0 + r >= a.M) break;
+        const float v = lin_act((part[0][r][n] + part[1][r][n]) + (part[2][r][n] + part[3][r][n]), a.act);
+        if (a.act && a.out_act == 1) ((uint16_t*)a.y)[(size_t)(m0 + r) * a.ldy + n] = f32_to_bf16_bits(v);
+        else ((float*)a.y)[(size_t)(m0 + r) * a.ldy + n] = v;
+    }
+}
+
 template <typename TA, bool DUAL>
 __global__ void __launch_bounds__(256) kf_lin_tile_kernel(LinArgs a) {
     const int g    = blockIdx.z;
@@ -425,6 +481,15 @@ bool skinny_shape(const LinArgs& a) { return a.N <= 128 && a.K >= 512 && a.M > k
 int dispatch_one(kf_ctx* ctx, const LinArgs& a, int act_f32) {
     const bool skinny = skinny_shape(a);
     if (skinny && a.K % 8 == 0 && a.ldx % 8 == 0 && (((uintptr_t)a.W0 | (uintptr_t)a.x) & 15) == 0 && (a.M + kSkR - 1) / kSkR <= 65535) {
+        if (!act_f32 && a.K % 32 == 0) {
+            const int nt = (a.N + 7) / 8, blocks = (a.M + 15) / 16;
+            if (nt <= 4) kf_lin_skinny_mma_kernel<4><<<blocks, 256, 0, ctx->stream>>>(a);
+            else if (nt <= 8) kf_lin_skinny_mma_kernel<8><<<blocks, 256, 0, ctx->stream>>>(a);
+            else if (nt <= 10) kf_lin_skinny_mma_kernel<10><<<blocks, 256, 0, ctx->stream>>>(a);
+            else kf_lin_skinny_mma_kernel<16><<<blocks, 256, 0, ctx->stream>>>(a);
+            KF_LAUNCH_CHECK(ctx);
+            return KF_OK;
+        }
         const dim3 grid((a.N + 8 * kSkC - 1) / (8 * kSkC), (a.M + kSkR - 1) / kSkR);
         if (act_f32) kf_lin_skinny_kernel<float><<<grid, 256, 0, ctx->stream>>>(a);
         else kf_lin_skinny_kernel<uint16_t><<<grid, 256, 0, ctx->stream>>>(a);

@@ -481,12 +481,12 @@ def test_routing_tables(ctx, M, X, P, top, groups, keep):
     assert (grp[off[X]:] == -1).all() and (row[off[X]:] == 0).all()
 
 
-@pytest.mark.parametrize("M, K", [(1, 128), (7, 50), (16, 128), (40, 128), (40, 50), (33, 640), (19, 1000), (21, 516)])
+@pytest.mark.parametrize("M, K", [(1, 128), (7, 50), (16, 128), (40, 128), (40, 50), (33, 640), (19, 1000), (21, 516), (130, 544)])
 @pytest.mark.parametrize("f32", [True, False])
 def test_batch_of_matmuls(ctx, M, K, f32):
     """kf_linear_batch: weights of different heights with inputs of their own, tanh on some, few rows and panels"""
     rs = np.random.RandomState(M + K)
-    N, act = [48, 5, 48, 16, 33], [0, 3, 0, 3, 0]
+    N, act = [48, 5, 128, 16, 75], [0, 3, 0, 3, 0]
     W = [grid(rs.randn(n, K) * K ** -0.5) for n in N]
     X = [grid(rs.randn(M, K)) for _ in N]
     wd = [ctx.array(bits(w)) for w in W]
